@@ -143,6 +143,14 @@ class ModelConfig:
 
     architecture: str
 
+    def needs_tensor_shapes(self) -> bool:
+        """True if a size of the model is given by a tensor's shape alone and is still open."""
+        return False
+
+    def with_tensor_shapes(self, shapes: Mapping[str, tuple]) -> "ModelConfig":
+        """This configuration with its open sizes read off the checkpoint's tensors (name -> shape)."""
+        return self
+
     def to_json_dict(self) -> dict:
         out = {}
         for f in fields(self):

@@ -135,6 +135,78 @@ rms_norm_vec_kernel(const float* __restrict__ x, const int* __restrict__ rows,
   }
 }
 
+// Layer norm with a bias: (x - mean) / sqrt(mean((x - mean)^2) + eps) * w + b (b may be null); the
+// deviations are taken from the mean first (two passes over the row, which stays in registers or in cache).
+template <typename TW, typename TO>
+__global__ void layer_norm_kernel(const float* __restrict__ x, const int* __restrict__ rows,
+                                  const TW* __restrict__ w, const TW* __restrict__ b, TO* __restrict__ out,
+                                  int hidden, float eps) {
+  __shared__ float scratch[33];
+  pdl_trigger();
+  pdl_wait();
+  const int r = blockIdx.x;
+  const float* src = x + (size_t)(rows ? rows[r] : r) * hidden;
+  float sum = 0.f;
+  for (int c = threadIdx.x; c < hidden; c += blockDim.x) sum += src[c];
+  const float mean = block_sum(sum, scratch) / (float)hidden;
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
+    const float d = src[c] - mean;
+    ss = fmaf(d, d, ss);
+  }
+  const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)hidden + eps);
+  TO* dst = out + (size_t)r * hidden;
+  for (int c = threadIdx.x; c < hidden; c += blockDim.x)
+    dst[c] = from_float<TO>(fmaf((src[c] - mean) * inv, to_float<TW>(w[c]), b ? to_float<TW>(b[c]) : 0.f));
+}
+
+template <typename TW, typename TO>
+__global__ void __launch_bounds__(kNormThreads)
+layer_norm_vec_kernel(const float* __restrict__ x, const int* __restrict__ rows, const TW* __restrict__ w,
+                      const TW* __restrict__ b, TO* __restrict__ out, int hidden, float eps) {
+  __shared__ float scratch[33];
+  pdl_trigger();
+  pdl_wait();
+  const int r = blockIdx.x;
+  const float* src = x + (size_t)(rows ? rows[r] : r) * hidden;
+  const int vecs = hidden >> 2;
+  float4 v[kNormItems];
+  float sum = 0.f;
+#pragma unroll
+  for (int i = 0; i < kNormItems; ++i) {
+    const int c = threadIdx.x + i * kNormThreads;
+    v[i] = c < vecs ? Vec4<float>::load(src + 4 * c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    sum += (v[i].x + v[i].y) + (v[i].z + v[i].w);
+  }
+  const float mean = block_sum(sum, scratch) / (float)hidden;
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < kNormItems; ++i) {
+    if (threadIdx.x + i * kNormThreads < vecs) {
+      v[i].x -= mean;
+      v[i].y -= mean;
+      v[i].z -= mean;
+      v[i].w -= mean;
+      ss = fmaf(v[i].x, v[i].x, ss);
+      ss = fmaf(v[i].y, v[i].y, ss);
+      ss = fmaf(v[i].z, v[i].z, ss);
+      ss = fmaf(v[i].w, v[i].w, ss);
+    }
+  }
+  const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)hidden + eps);
+  TO* dst = out + (size_t)r * hidden;
+#pragma unroll
+  for (int i = 0; i < kNormItems; ++i) {
+    const int c = threadIdx.x + i * kNormThreads;
+    if (c < vecs) {
+      const float4 g = Vec4<TW>::load(w + 4 * c);
+      const float4 a = b ? Vec4<TW>::load(b + 4 * c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      Vec4<TO>::store(dst + 4 * c, make_float4(fmaf(v[i].x * inv, g.x, a.x), fmaf(v[i].y * inv, g.y, a.y),
+                                               fmaf(v[i].z * inv, g.z, a.z), fmaf(v[i].w * inv, g.w, a.w)));
+    }
+  }
+}
+
 // ---------------------------------------------------------------------------
 // SwiGLU on stacked [gate | up] rows: out = gate / (1 + exp(-gate)) * up
 // (crates/leone/src/cpu.rs:903-905; ie_cuda.cu:2864-2874).
@@ -152,11 +224,13 @@ __global__ void swiglu_kernel(const T* __restrict__ gate_up, T* __restrict__ out
 }
 
 // The gated layer with its gate's shape as parameters:
-//   g' = min(g, limit), u' = clamp(u, -limit, limit), out = g' * sigmoid(slope * g') * (u' + shift)
-// (limit = +inf: no clamping).  slope 1, no limit and shift 0 are SwiGLU.
+//   g' = min(g, limit), u' = clamp(u, -limit, limit),
+//   out = g' * sigmoid(slope * g' * (1 + cubic * g'^2)) * (u' + shift)
+// (limit = +inf: no clamping).  slope 1, no limit, shift and cubic 0 are SwiGLU; slope 2 sqrt(2/pi) with
+// cubic 0.044715 is gelu's tanh form (z/2 (1 + tanh y) = z sigmoid(2y)).
 template <typename T>
 __global__ void gated_act_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int n, int inter, float slope,
-                                 float limit, float shift) {
+                                 float limit, float shift, float cubic) {
   pdl_trigger();
   pdl_wait();
   const size_t total = (size_t)n * inter;
@@ -165,7 +239,7 @@ __global__ void gated_act_kernel(const T* __restrict__ gate_up, T* __restrict__ 
     const size_t row = i / inter, col = i - row * inter;
     const float g = fminf(to_float<T>(gate_up[row * 2 * inter + col]), limit);
     const float u = fminf(fmaxf(to_float<T>(gate_up[row * 2 * inter + inter + col]), -limit), limit);
-    out[i] = from_float<T>(g / (1.f + expf(-slope * g)) * (u + shift));
+    out[i] = from_float<T>(g / (1.f + expf(-slope * g * fmaf(cubic * g, g, 1.f))) * (u + shift));
   }
 }
 
@@ -629,6 +703,30 @@ extern "C" int leone_rms_norm(const float* x, const int* rows, const void* w, in
   return kRefusedDtype;
 }
 
+// w and b (b may be null) in `w_dtype`.
+extern "C" int leone_layer_norm(const float* x, const int* rows, const void* w, const void* b, int w_dtype, void* out,
+                                int out_dtype, int n_out, int hidden, float eps, cudaStream_t stream) {
+  if (n_out <= 0) return 0;
+  if (hidden <= 0) return kRefusedSize;
+  const int threads = hidden >= 2048 ? 512 : (hidden >= 512 ? 256 : 128);
+  const bool vec = (hidden % 4) == 0 && hidden >= 512 && hidden <= kNormThreads * kNormItems * 4 &&
+                   (((uintptr_t)x | (uintptr_t)w | (uintptr_t)b | (uintptr_t)out) & 15) == 0;
+#define LAUNCH(TW, TO)                                                                                       \
+  {                                                                                                          \
+    if (vec)                                                                                                 \
+      return launch_kernel(layer_norm_vec_kernel<TW, TO>, dim3(n_out), dim3(kNormThreads), 0, stream, x,     \
+                           rows, (const TW*)w, (const TW*)b, (TO*)out, hidden, eps);                         \
+    return launch_kernel(layer_norm_kernel<TW, TO>, dim3(n_out), dim3(threads), 0, stream, x, rows,          \
+                         (const TW*)w, (const TW*)b, (TO*)out, hidden, eps);                                 \
+  }
+  if (w_dtype == 0 && out_dtype == 0) LAUNCH(float, float);
+  if (w_dtype == 0 && out_dtype == 1) LAUNCH(float, __nv_bfloat16);
+  if (w_dtype == 1 && out_dtype == 0) LAUNCH(__nv_bfloat16, float);
+  if (w_dtype == 1 && out_dtype == 1) LAUNCH(__nv_bfloat16, __nv_bfloat16);
+#undef LAUNCH
+  return kRefusedDtype;
+}
+
 extern "C" int leone_swiglu(int dtype, const void* gate_up, void* out, int n, int inter,
                             cudaStream_t stream) {
   if (n <= 0) return 0;
@@ -645,17 +743,17 @@ extern "C" int leone_swiglu(int dtype, const void* gate_up, void* out, int n, in
 }
 
 extern "C" int leone_gated_act(int dtype, const void* gate_up, void* out, int n, int inter, float slope, float limit,
-                               float shift, cudaStream_t stream) {
+                               float shift, float cubic, cudaStream_t stream) {
   if (n <= 0) return 0;
   if (inter <= 0 || !(limit > 0.f)) return kRefusedSize;
   const size_t total = (size_t)n * inter;
   const int blocks = (int)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
   if (dtype == 0)
     return launch_kernel(gated_act_kernel<float>, dim3(blocks), dim3(256), 0, stream, (const float*)gate_up,
-                         (float*)out, n, inter, slope, limit, shift);
+                         (float*)out, n, inter, slope, limit, shift, cubic);
   if (dtype == 1)
     return launch_kernel(gated_act_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream,
-                         (const __nv_bfloat16*)gate_up, (__nv_bfloat16*)out, n, inter, slope, limit, shift);
+                         (const __nv_bfloat16*)gate_up, (__nv_bfloat16*)out, n, inter, slope, limit, shift, cubic);
   return kRefusedDtype;
 }
 

@@ -59,18 +59,19 @@ struct GemmParams {
   int norm_in_parts;
   float norm_eps;
   int l2_ahead;      // k-blocks of weights past the early stages that the producer asks the L2 for
-  // The gate's shape of epilogue 3: g' sigmoid(slope g') (u' + shift) with g' = min(g, limit) and
-  // u' = clamp(u, -limit, limit).  gate_plain: slope 1, no limit, shift 0 (SwiGLU).
+  // The gate's shape of epilogue 3: g' sigmoid(slope g' (1 + cubic g'^2)) (u' + shift) with g' = min(g, limit)
+  // and u' = clamp(u, -limit, limit).  gate_plain: slope 1, no limit, shift and cubic 0 (SwiGLU).
   int gate_plain;
-  float gate_slope, gate_limit, gate_shift;
+  float gate_slope, gate_limit, gate_shift, gate_cubic;
 };
 
-// Host side: the four gate fields from an optional {slope, limit, shift} (null: SwiGLU).
+// Host side: the gate fields from an optional {slope, limit, shift, cubic} (null: SwiGLU).
 inline void set_gate_shape(GemmParams& p, const float* shape) {
   p.gate_plain = shape == nullptr ? 1 : 0;
   p.gate_slope = shape == nullptr ? 1.f : shape[0];
   p.gate_limit = shape == nullptr ? INFINITY : shape[1];
   p.gate_shift = shape == nullptr ? 0.f : shape[2];
+  p.gate_cubic = shape == nullptr ? 0.f : shape[3];
 }
 
 __device__ __forceinline__ long long global_ns() {
@@ -103,7 +104,8 @@ __device__ __forceinline__ float gate_mul(const GemmParams& p, float g, float u)
   if (p.gate_plain) return silu_mul(g, u);
   g = fminf(g, p.gate_limit);
   u = fminf(fmaxf(u, -p.gate_limit), p.gate_limit);
-  return __fdividef(g, 1.f + __expf(-p.gate_slope * g)) * (u + p.gate_shift);
+  const float z = p.gate_slope * g * fmaf(p.gate_cubic * g, g, 1.f);
+  return __fdividef(g, 1.f + __expf(-z)) * (u + p.gate_shift);
 }
 
 // Swapped orientation: the thread that owns weight row n finishes NC token columns

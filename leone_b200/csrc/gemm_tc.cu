@@ -712,7 +712,7 @@ extern "C" int leone_gemm_tc_cluster_capacity_token_major(int splits) {
 // x: [m, k] bf16 (row stride ldx), w: [n, k] bf16 (row stride ldw), out: [m, n] (row stride ldc).
 // epilogue 0: bf16 out; 1: fp32 out; 2: fp32 out = acc + residual (same layout as out);
 // 3: w holds interleaved gate/up rows, out is bf16 [m, n/2] = silu(gate) * up; gate_shape (host
-// floats {slope, limit, shift}, or null) gives the gate another shape (see GemmParams).
+// floats {slope, limit, shift, cubic}, or null) gives the gate another shape (see GemmParams).
 // The first `full_tiles` tiles (in the kernel's tile order) are computed whole; the others have K
 // split `splits` ways.  splits > 1 needs `workspace` (fp32) and zeroed `counters` of the sizes
 // leone_gemm_tc_scratch gives for (tiles - full_tiles).  More than 256 tokens are never split.

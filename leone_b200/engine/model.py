@@ -118,13 +118,12 @@ class Model:
         """Gives every part its tensors; ``tensors`` is emptied on the way, so a source that a
         part fused into a copy of its own (q/k/v stacked, gate/up interleaved) is freed as soon
         as that part is loaded."""
-        s = self.spec
         self.embedding.load({w.name: tensors.pop(w.name) for w in self.embedding.weight_specs()})
         for holder in self._holders:
             holder.load(tensors)
         for _, part in self._injection_parts:
             part.load({w.name: tensors.pop(w.name) for w in part.weight_specs()})
-        self.final_norm.load({s.final_norm_name: tensors.pop(s.final_norm_name)})
+        self.final_norm.load({w.name: tensors.pop(w.name) for w in self.final_norm.weight_specs()})
         self.head.load({w.name: tensors.pop(w.name) for w in self.head.weight_specs()}, self.embedding)
 
     # -- cache needs ------------------------------------------------------------------

@@ -190,6 +190,23 @@ class CudaOps:
                                         _ptr(out), _dt(out.dtype), n_out, hidden, c_float(eps),
                                         self._stream()), "rms_norm")
 
+    def layer_norm(self, x, weight, bias, out, eps, rows=None):
+        """``out = (x - mean) / sqrt(mean((x - mean)^2) + eps) * weight + bias`` (``bias`` may be None) of
+        the fp32 rows of ``x`` (``rows``: which of them)."""
+        n_out, hidden = out.shape
+        _need(x.dtype == torch.float32 and x.is_contiguous() and x.shape[1] == hidden,
+              "layer_norm input must be contiguous fp32 [*, hidden]")
+        _need(weight.numel() == hidden and weight.is_contiguous() and out.is_contiguous()
+              and (bias is None or (bias.numel() == hidden and bias.dtype == weight.dtype and bias.is_contiguous())),
+              "layer_norm weight/bias/output shape")
+        if rows is not None:
+            _need(rows.dtype == torch.int32 and rows.numel() == n_out, "layer_norm rows must be int32")
+        else:
+            _need(x.shape[0] >= n_out, "layer_norm input has fewer rows than the output")
+        self.launches += 1
+        _check(self.core.leone_layer_norm(_ptr(x), _ptr(rows), _ptr(weight), _ptr(bias), _dt(weight.dtype), _ptr(out),
+                                          _dt(out.dtype), n_out, hidden, c_float(eps), self._stream()), "layer_norm")
+
     def _gemm_simt(self, x, w, out, epilogue, residual):
         m, k = x.shape
         n = w.shape[0]
@@ -265,13 +282,13 @@ class CudaOps:
 
     def linear_swiglu(self, x, w_gate_up: PreparedMatrix, out, norm_in=None, gate_shape=None):
         """``out = silu(x @ gate.T) * (x @ up.T)`` for a matrix from ``prepare_gate_up``.
-        ``gate_shape = (slope, limit, shift)``: ``g' sigmoid(slope g') (u' + shift)`` with
-        ``g' = min(g, limit)``, ``u' = clamp(u, -limit, limit)`` (``limit`` may be ``inf``)."""
+        ``gate_shape = (slope, limit, shift, cubic)``: ``g' sigmoid(slope g' (1 + cubic g'^2)) (u' + shift)``
+        with ``g' = min(g, limit)``, ``u' = clamp(u, -limit, limit)`` (``limit`` may be ``inf``)."""
         m = x.shape[0]
         inter = w_gate_up.out_features // 2
         _need(out.shape == (m, inter) and out.dtype == x.dtype and out.is_contiguous(),
               "linear_swiglu: output shape")
-        _need(gate_shape is None or (len(gate_shape) == 3 and gate_shape[1] > 0), "linear_swiglu: gate shape")
+        _need(gate_shape is None or (len(gate_shape) == 4 and gate_shape[1] > 0), "linear_swiglu: gate shape")
         if m == 0:
             return
         if norm_in is not None:
@@ -291,9 +308,9 @@ class CudaOps:
             _check(self.core.leone_swiglu(_dt(x.dtype), _ptr(scratch), _ptr(out), m, inter,
                                           self._stream()), "swiglu")
         else:
-            slope, limit, shift = gate_shape
+            slope, limit, shift, cubic = gate_shape
             _check(self.core.leone_gated_act(_dt(x.dtype), _ptr(scratch), _ptr(out), m, inter, c_float(slope),
-                                             c_float(limit), c_float(shift), self._stream()), "gated_act")
+                                             c_float(limit), c_float(shift), c_float(cubic), self._stream()), "gated_act")
 
     def convert(self, src, out):
         """``out = src`` elementwise, ``src`` fp32, ``out`` fp32 or the run dtype (same shape)."""
@@ -540,6 +557,41 @@ class CudaOps:
             _dt(proj.dtype), _ptr(proj), proj.stride(0), q_off, k_off, v_off, _ptr(out), out.stride(0), _ptr(state),
             _ptr(ctx.q_start), _ptr(ctx.slot_ids), _ptr(decay), ctx.n_seqs, heads, dim, vdim, state.shape[0], chunk,
             n_chunks, _ptr(chunk_state), _ptr(ctx.status), self._stream()), "linear_attention")
+
+    def gated_linear_attention(self, ctx, proj, gated, state, w2, w2_bias, norm_w, heads, dim, vdim, rank, tau, q_scale,
+                               eps, q_off, k_off, v_off, u_off, gate_off, chunk=0, act="silu"):
+        """The recurrence with a decay per key channel over the step's tokens, every head's output normed and
+        gated (``csrc/gated_linear_attention.cu``).  ``proj``: fp32 rows with q, k, v, the decay's low-rank
+        part u and the gate at their offsets; ``w2``: fp32 ``[rank, heads * dim]`` and ``w2_bias`` make the
+        decay's logits of u; ``norm_w``: fp32 ``[vdim]``; ``gated``: ``[n, heads * vdim]`` in the run dtype.
+        ``chunk`` > 0: prompt portions are cut into chunks of that many tokens that run side by side."""
+        n = proj.shape[0]
+        hv = heads * vdim
+        _need(proj.dtype == torch.float32 and proj.stride(1) == 1 and gated.shape == (n, hv) and gated.stride(1) == 1,
+              "gated_linear_attention layout")
+        _need(state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (heads, dim, vdim)
+              and w2.dtype == torch.float32 and w2.is_contiguous() and tuple(w2.shape) == (rank, heads * dim)
+              and w2_bias.dtype == torch.float32 and w2_bias.numel() == heads * dim
+              and norm_w.dtype == torch.float32 and norm_w.numel() == vdim, "gated_linear_attention state/constants")
+        _need(max(q_off, k_off) + heads * dim <= proj.shape[1] and max(v_off, gate_off) + hv <= proj.shape[1]
+              and u_off + rank <= proj.shape[1] and act in ("sigmoid", "silu"), "gated_linear_attention columns")
+        n_chunks, chunk_state, chunk_decay = 0, None, None
+        if chunk > 0:
+            n_chunks = int(sum(-(-int(q) // chunk) for q in ctx.q_lens))
+            chunk_state = self._scratch("gla_chunk_state", n_chunks, heads * dim * vdim, torch.float32)
+            chunk_decay = self._scratch("gla_chunk_decay", n_chunks, heads * dim, torch.float32)
+        # a head wider than a block's columns is normed and gated by a kernel of its own
+        whole = vdim <= (128 if dim <= 128 else 64 if dim <= 256 else 32)
+        o = None if whole else self._scratch("gla_out", n, hv, torch.float32)
+        self.launches += 1 if chunk == 0 else 3
+        _check(self.mixers.leone_gla(
+            _dt(gated.dtype), _ptr(proj), proj.stride(0), q_off, k_off, v_off, u_off, gate_off, _ptr(w2), _ptr(w2_bias), rank,
+            c_float(1.0 / tau), c_float(q_scale), _ptr(o), 0 if o is None else o.stride(0), _ptr(gated) if whole else c_void_p(0),
+            gated.stride(0), _ptr(norm_w), 1 if act == "silu" else 0, c_float(eps), _ptr(state), _ptr(ctx.q_start),
+            _ptr(ctx.slot_ids), ctx.n_seqs, heads, dim, vdim, state.shape[0], chunk, n_chunks, _ptr(chunk_state),
+            _ptr(chunk_decay), _ptr(ctx.status), self._stream()), "gated_linear_attention")
+        if not whole:
+            self.group_gate_norm(o, norm_w, proj[:, gate_off:gate_off + hv], gated, eps, heads, vdim, act=act)
 
     def gate_norm(self, o, weight, gate, out, eps):
         """``out = rms_norm(o) * weight * sigmoid(gate)``; ``o`` fp32, ``gate`` a column slice."""

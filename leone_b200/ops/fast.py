@@ -310,8 +310,8 @@ class FastKernels:
         no = (None, None, None, 0) if norm_out is None else \
             (_ptr(norm_out[0]), _ptr(norm_out[1]), _ptr(norm_out[2]), norm_out[0].stride(0))
         ni = (None, 0, c_float(0.0)) if norm_in is None else (_ptr(norm_in[0]), int(norm_in[1]), c_float(norm_in[2]))
-        # the gate's shape of the gated epilogue: three host floats, or null for SwiGLU
-        gs = None if gate_shape is None else (c_float * 3)(*[float(v) for v in gate_shape])
+        # the gate's shape of the gated epilogue: four host floats, or null for SwiGLU
+        gs = None if gate_shape is None else (c_float * 4)(*[float(v) for v in gate_shape])
         if pairs:
             # pairs of SMs on tiles of 256 tokens (gemm_pair.cu)
             code = self.lib.leone_gemm_pair(_ptr(x), _ptr(w), _ptr(out), _ptr(residual), m, n_rows, k,

@@ -25,6 +25,8 @@ counted from position 0 of the sequence).
 ``weights``: how scores become weights: ``"softmax"``; ``"softmax_plus_one"`` (``exp(s_j) / (1 +
 sum exp(s_j))``: one more member of score 0 without a value); ``"sigmoid"`` (``sigmoid(s_j +
 b_head)`` for every seen key on its own, nothing normalised; ``b`` is the tensor ``bias_name``).
+``gate_name``: an elementwise output gate: the heads' outputs, concatenated, times ``sigmoid(W_g x)`` (``W_g``:
+``[heads * value_head_dim, hidden]``, rows of the fused input product) before ``W_o``.
 ``qk_norm = "whole"``: one RMS norm over all of a token's query heads together (weight
 ``[heads * head_dim]``, multiplied directly) and one over its key heads, before rotation.
 A position encoding that offers ``frequencies()`` instead of a table (``rotary_computed``): the
@@ -84,6 +86,7 @@ class Attention(Mixer):
         self.mixed = bool(self.temp_name or self.mix_name or self.sink_name or self.score_cap)
         if self.mixed and self.weights != "softmax":
             raise ValueError("attention: temperature, cap, mixing and sink go with softmax weights")
+        self.gate_name = params.get("gate_name")
         self.scale = float(params.get("scale", 1.0 / math.sqrt(self.d)))
         pe_name = params.get("position_encoding")
         self.pos = (position_encodings or {}).get(pe_name) if pe_name else None
@@ -94,9 +97,13 @@ class Attention(Mixer):
         self.k_norm_name = params.get("k_norm_name", "k_norm.weight")
         self.w_qkv = self.w_o = self.q_norm_w = self.k_norm_w = None
         self.qkv_cols = (self.n_q + self.n_kv) * self.d + self.n_kv * self.dv
+        # the gate's rows of the input product start a padded row after the values
+        self.gate_off = -(-self.qkv_cols // 16) * 16
+        self.gate_rows = self.n_q * self.dv if self.gate_name else 0
+        self.in_cols = -(-(self.gate_off + self.gate_rows) // 16) * 16 if self.gate_name else self.qkv_cols
         # the layer as the reference has it runs on the kernels tuned for it; anything else on the general ones
         self.general = (self.dv != self.d or self.mask == "chunk" or self.weights != "softmax" or self.norm_whole
-                        or self.mixed or (self.pos is not None and hasattr(self.pos, "frequencies")))
+                        or self.mixed or bool(self.gate_name) or (self.pos is not None and hasattr(self.pos, "frequencies")))
         if self.general and self.pos is not None and not hasattr(self.pos, "frequencies"):
             raise ValueError("attention: the general kernels take a position encoding that offers its frequencies")
 
@@ -105,6 +112,8 @@ class Attention(Mixer):
                  WeightSpec(self.names["k"], (self.n_kv * self.d, self.hidden)),
                  WeightSpec(self.names["v"], (self.n_kv * self.dv, self.hidden)),
                  WeightSpec(self.names["o"], (self.hidden, self.n_q * self.dv))]
+        if self.gate_name:
+            specs.append(WeightSpec(self.gate_name, (self.gate_rows, self.hidden)))
         if self.qk_norm:
             nq, nk = (self.n_q * self.d, self.n_kv * self.d) if self.norm_whole else (self.d, self.d)
             specs += [WeightSpec(self.q_norm_name, (nq,), role="norm", std=0.1),
@@ -120,9 +129,13 @@ class Attention(Mixer):
         return specs
 
     def load(self, tensors):
-        stacked = torch.cat([tensors[self.names["q"]], tensors[self.names["k"]],
-                             tensors[self.names["v"]]], dim=0).contiguous()
-        self.w_qkv = self.rt.ops.prepare_matrix(stacked)
+        rows = [tensors[self.names["q"]], tensors[self.names["k"]], tensors[self.names["v"]]]
+        if self.gate_name:
+            def zeros(count):
+                return torch.zeros((count, self.hidden), dtype=rows[0].dtype, device=rows[0].device)
+            rows += [zeros(self.gate_off - self.qkv_cols), tensors[self.gate_name],
+                     zeros(self.in_cols - self.gate_off - self.gate_rows)]
+        self.w_qkv = self.rt.ops.prepare_matrix(torch.cat(rows, dim=0).contiguous())
         self.w_o = self.rt.ops.prepare_matrix(tensors[self.names["o"]])
         self.q_norm_f32 = self.k_norm_f32 = None
         if self.qk_norm:
@@ -138,13 +151,13 @@ class Attention(Mixer):
         self.sink = tensors[self.sink_name].float().contiguous() if self.sink_name else None
 
     def weight_bytes(self):
-        return (self.qkv_cols * self.hidden + self.hidden * self.n_q * self.dv) * self.rt.dtype.itemsize
+        return (self.in_cols * self.hidden + self.hidden * self.n_q * self.dv) * self.rt.dtype.itemsize
 
     def scratch_bytes(self, max_tokens):
-        return max_tokens * (self.qkv_cols + self.n_q * self.dv) * self.rt.dtype.itemsize
+        return max_tokens * (self.in_cols + self.n_q * self.dv) * self.rt.dtype.itemsize
 
     def load_transient_bytes(self):
-        return self.qkv_cols * self.hidden * self.rt.dtype.itemsize       # q, k, v beside their stacked copy
+        return self.in_cols * self.hidden * self.rt.dtype.itemsize       # q, k, v beside their stacked copy
 
     def cache_request(self):
         return PagedKV(self.n_kv, self.d, self.window, value_head_dim=self.dv)
@@ -166,7 +179,7 @@ class Attention(Mixer):
     def forward(self, ctx, cache, x, hidden, then=None, fresh=False):
         rt = self.rt
         n = hidden.shape[0]
-        qkv = rt.buffer("qkv", n, self.qkv_cols, rt.dtype)
+        qkv = rt.buffer("qkv", n, self.in_cols, rt.dtype)
         if isinstance(x, DeferredNorm):
             if x.ready and rt.ops.linear_fuses_norm(n, self.w_qkv):
                 rt.ops.linear(x.xn, self.w_qkv, qkv, norm_in=x)          # the norm's factor in the epilogue
@@ -175,7 +188,8 @@ class Attention(Mixer):
         else:
             rt.ops.linear(x, self.w_qkv, qkv)
         if self.general:
-            self._forward_general(ctx, cache, qkv, hidden, then, fresh)
+            gate = qkv[:, self.gate_off:self.gate_off + self.gate_rows] if self.gate_name else None
+            self._forward_general(ctx, cache, qkv[:, :self.qkv_cols], gate, hidden, then, fresh)
             return
         table, rotary_dim, pairing = None, 0, None
         if self.pos is not None:
@@ -215,7 +229,7 @@ class Attention(Mixer):
                          self.window, cache)
         self._out_proj(attn, hidden, then, fresh)
 
-    def _forward_general(self, ctx, cache, qkv, hidden, then, fresh=False):
+    def _forward_general(self, ctx, cache, qkv, gate, hidden, then, fresh=False):
         """Masks, weight rules, norms and widths beyond the reference's layer: one kernel norms and
         rotates q and k in fp32 and writes the new keys and values into their pages, one does the
         attention over the pages.  A layer that is causal softmax attention with equal key and
@@ -239,4 +253,6 @@ class Attention(Mixer):
         else:
             ops.attention_masked(ctx, qkv, attn, self.n_q, self.n_kv, self.d, self.dv, self.scale, self.mask,
                                  int(size or 0), self.weights, self.bias, cache)
+        if gate is not None:
+            ops.gate_rows(attn, gate, "sigmoid")
         self._out_proj(attn, hidden, then, fresh)

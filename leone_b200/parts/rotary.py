@@ -55,10 +55,29 @@ class RotaryAdjacent(RotaryHalfSplit):
     pairing = "adjacent"
 
 
+def wavelength_scaled(freqs, factor: float, low: float, high: float, original: float):
+    """Frequencies judged by their wavelength ``l = 2 pi / f``: kept where ``l < original / high``, divided by
+    ``factor`` where ``l > original / low``, and between the two ``(1 - s) f / factor + s f`` with
+    ``s = (original / l - low) / (high - low)``."""
+    import math
+    out = []
+    for f in freqs:
+        wave = 2.0 * math.pi / f
+        if wave < original / high:
+            out.append(f)
+        elif wave > original / low:
+            out.append(f / factor)
+        else:
+            s = (original / wave - low) / (high - low) if high > low else 1.0
+            out.append((1.0 - s) * f / factor + s * f)
+    return out
+
+
 def scaled_frequencies(dims: int, base: float, scaling=None):
-    """Per pair ``i`` the frequency ``f_i = base^(-2i/dims)``, blended by YaRN if ``scaling``
-    (a mapping with ``factor``, ``original``, ``fast``, ``slow``) is given, and the factor that
-    multiplies cos and sin.
+    """Per pair ``i`` the frequency ``f_i = base^(-2i/dims)``, rescaled if ``scaling`` is given, and the
+    factor that multiplies cos and sin.  ``scaling``: a mapping whose ``kind`` is ``"wavelength"`` (``factor``,
+    ``low``, ``high``, ``original``; see :func:`wavelength_scaled`; the factor is 1) or ``"yarn"`` (the default:
+    ``factor``, ``original``, ``fast``, ``slow``).
 
     YaRN (Peng et al., "YaRN: Efficient Context Window Extension of Large Language Models"): a
     pair that turns more than ``fast`` times within ``original`` positions keeps its frequency,
@@ -72,6 +91,11 @@ def scaled_frequencies(dims: int, base: float, scaling=None):
     freqs = [float(base) ** (-2.0 * i / dims) for i in range(half)]
     if not scaling:
         return freqs, 1.0
+    kind = scaling.get("kind", "yarn")
+    if kind == "wavelength":
+        return wavelength_scaled(freqs, *(float(scaling[k]) for k in ("factor", "low", "high", "original"))), 1.0
+    if kind != "yarn":
+        raise ValueError(f"rotary scaling '{kind}' is not one of yarn, wavelength")
     factor, original = float(scaling["factor"]), float(scaling["original"])
 
     def idx(turns):
@@ -91,8 +115,8 @@ def scaled_frequencies(dims: int, base: float, scaling=None):
 class RotaryComputed(PositionEncoding):
     """A rotary encoding without a table and so without a limit on positions: it offers its
     per-pair frequencies (fp32) and a magnitude, and the kernel that applies it forms the angle
-    ``position * frequency`` and its cos and sin in fp32 itself.  ``scaling``: YaRN constants or
-    ``None``.  ``pairing``: ``"adjacent"`` (pair i = elements 2i, 2i+1) or ``"half_split"``."""
+    ``position * frequency`` and its cos and sin in fp32 itself.  ``scaling``: constants of
+    :func:`scaled_frequencies` (YaRN, or by wavelength) or ``None``.  ``pairing``: ``"adjacent"`` (pair i = elements 2i, 2i+1) or ``"half_split"``."""
 
     def __init__(self, params, rt):
         super().__init__(params, rt)

@@ -6,11 +6,14 @@ matrices are stacked row-wise at load time so one product feeds both
 (the reference pairs them in one launch too, ie_cuda.cu:1896-1931).
 
 The gate's shape is this part's own parameters, for gated layers of the same family:
-``y = g' * sigmoid(gate_slope * g') * (u' + up_shift)`` with ``g' = min(g, limit)`` and
-``u' = clamp(u, -limit, limit)``.  The defaults (``gate_slope = 1``, no ``limit``, ``up_shift = 0``)
-are SwiGLU.
+``y = g' * sigmoid(gate_slope * g' * (1 + gate_cubic * g'^2)) * (u' + up_shift)`` with ``g' = min(g, limit)``
+and ``u' = clamp(u, -limit, limit)``.  The defaults (``gate_slope = 1``, no ``limit``, ``up_shift`` and
+``gate_cubic`` 0) are SwiGLU.  ``activation = "gelu_tanh"`` sets the slope and the cubic term to gelu's tanh form
+(GeGLU): ``z/2 (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))) = z sigmoid(2 sqrt(2/pi) z (1 + 0.044715 z^2))``.
 """
 from __future__ import annotations
+
+import math
 
 from ..registry import FEED_FORWARDS
 from .base import DeferredNorm, FeedForward, WeightSpec
@@ -31,12 +34,19 @@ class SwiGLU(FeedForward):
         self.down_name = params.get("down_name", "down_proj.weight")
         self.w_gate_up = None
         self.w_down = None
-        slope, limit, shift = float(params.get("gate_slope", 1.0)), params.get("limit"), float(params.get("up_shift", 0.0))
+        activation = params.get("activation", "silu")
+        if activation not in ("silu", "gelu_tanh"):
+            raise ValueError(f"a gated layer's activation is silu or gelu_tanh, not '{activation}'")
+        if activation == "gelu_tanh" and ("gate_slope" in params or "gate_cubic" in params):
+            raise ValueError("a gated layer's activation gelu_tanh sets the gate's slope and cubic term itself")
+        slope, cubic = (2.0 * math.sqrt(2.0 / math.pi), 0.044715) if activation == "gelu_tanh" else \
+            (float(params.get("gate_slope", 1.0)), float(params.get("gate_cubic", 0.0)))
+        limit, shift = params.get("limit"), float(params.get("up_shift", 0.0))
         if limit is not None and not float(limit) > 0.0:
             raise ValueError(f"a gated layer's limit must be positive, got {limit}")
-        # None: plain SwiGLU (the kernels' default); else (slope, limit, shift) with limit = inf for none
-        self.gate_shape = None if (slope == 1.0 and limit is None and shift == 0.0) else \
-            (slope, float("inf") if limit is None else float(limit), shift)
+        # None: plain SwiGLU (the kernels' default); else (slope, limit, shift, cubic) with limit = inf for none
+        self.gate_shape = None if (slope == 1.0 and limit is None and shift == 0.0 and cubic == 0.0) else \
+            (slope, float("inf") if limit is None else float(limit), shift, cubic)
 
     def weight_specs(self):
         return [WeightSpec(self.gate_name, (self.inter, self.hidden)),

@@ -83,10 +83,22 @@ ARCHITECTURES = ArchitectureRegistry()
 
 
 def config_from_folder(folder: str):
-    """Read ``folder/config.json`` into the typed configuration of its architecture."""
-    from .config.base import architecture_name, read_config_json
+    """Read ``folder/config.json`` into the typed configuration of its architecture; sizes that only a
+    tensor's shape gives come from the checkpoint beside it, if there is one."""
+    from .config.base import read_config_json
     raw = read_config_json(folder)
-    return config_from_dict(raw)
+    config = config_from_dict(raw)
+    if config.needs_tensor_shapes():
+        from .weights.safetensors import Checkpoint, SafetensorsError
+        try:
+            ckpt = Checkpoint(folder)
+        except SafetensorsError:
+            return config
+        try:
+            config = config.with_tensor_shapes({name: tuple(e.shape) for name, e in ckpt.entries.items()})
+        finally:
+            ckpt.close()
+    return config
 
 
 def config_from_dict(raw: dict):

@@ -44,6 +44,12 @@ class EmulatedOps:
         ms = (src * src).mean(dim=-1, keepdim=True)
         out.copy_((src * weight.float() * torch.rsqrt(ms + eps)).to(out.dtype))
 
+    def layer_norm(self, x, weight, bias, out, eps, rows=None):
+        src = (x if rows is None else x[rows.long()]).float()
+        d = src - src.mean(dim=-1, keepdim=True)
+        y = d * torch.rsqrt((d * d).mean(dim=-1, keepdim=True) + eps) * weight.float()
+        out.copy_((y if bias is None else y + bias.float()).to(out.dtype))
+
     def linear(self, x, w, out, residual=None):
         y = x.float() @ w.float().t()
         if residual is not None:
@@ -56,9 +62,9 @@ class EmulatedOps:
         if self.dtype != torch.float32:
             y = y.to(self.dtype).float()
         g, u = y[:, :inter], y[:, inter:]
-        slope, limit, shift = gate_shape or (1.0, float("inf"), 0.0)
+        slope, limit, shift, cubic = gate_shape or (1.0, float("inf"), 0.0, 0.0)
         g, u = torch.clamp(g, max=limit), torch.clamp(u, min=-limit, max=limit)
-        out.copy_((g / (1.0 + torch.exp(-slope * g)) * (u + shift)).to(out.dtype))
+        out.copy_((g / (1.0 + torch.exp(-slope * g * (1.0 + cubic * g * g))) * (u + shift)).to(out.dtype))
 
     def convert(self, src, out):
         out.copy_(src.to(out.dtype))
@@ -162,7 +168,7 @@ class EmulatedOps:
 
     def attention(self, ctx, qkv, out, n_q, n_kv, d, scale, window, cache):
         n = qkv.shape[0]
-        q = qkv.float().view(n, n_q + 2 * n_kv, d)[:, :n_q]
+        q = qkv.float().reshape(n, n_q + 2 * n_kv, d)[:, :n_q]
         g = n_q // n_kv
         pt = cache.page_tokens
         res = torch.zeros(n, n_q, d)
@@ -485,6 +491,23 @@ class EmulatedOps:
                 st = st + k[:, :, None] * u[:, None, :]
                 out[t] = torch.einsum("hdv,hd->hv", st, q).reshape(-1)
             state[slot] = st
+
+    def gated_linear_attention(self, ctx, proj, gated, state, w2, w2_bias, norm_w, heads, dim, vdim, rank, tau, q_scale,
+                               eps, q_off, k_off, v_off, u_off, gate_off, chunk=0, act="silu"):
+        n, hd, hv = proj.shape[0], heads * dim, heads * vdim
+        z = proj[:, u_off:u_off + rank] @ w2 + w2_bias
+        alpha = torch.exp(torch.nn.functional.logsigmoid(z) / tau).view(n, heads, dim)
+        q = (proj[:, q_off:q_off + hd] * q_scale).view(n, heads, dim)
+        k, v = proj[:, k_off:k_off + hd].view(n, heads, dim), proj[:, v_off:v_off + hv].view(n, heads, vdim)
+        o = torch.zeros(n, hv)
+        bounds, slots = ctx.q_start.tolist(), ctx.slot_ids.tolist()
+        for s, slot in enumerate(slots):
+            st = state[slot]
+            for t in range(bounds[s], bounds[s + 1]):
+                st = alpha[t][:, :, None] * st + k[t][:, :, None] * v[t][:, None, :]
+                o[t] = torch.einsum("hdv,hd->hv", st, q[t]).reshape(-1)
+            state[slot] = st
+        self.group_gate_norm(o, norm_w, proj[:, gate_off:gate_off + hv], gated, eps, heads, vdim, act=act)
 
     def group_gate_norm(self, o, weight, gate, out, eps, heads, vdim, act="sigmoid"):
         n = o.shape[0]
