@@ -470,6 +470,19 @@ def _ziginex_shape(width: int, layers: int, heads: int, experts: int, top: int, 
             "layers": out}
 
 
+def _kakirax_shape(width: int, layers: int, heads: int, ff: int, vocab: int) -> dict:
+    """Layer sizes that resemble a real model's: three gated-linear-attention layers to every attention layer
+    (four query heads to a key/value head, rotation scaled by wavelength), a dense gated layer everywhere."""
+    attn = {"heads": heads, "kv_heads": max(heads // 4, 1), "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+            "rot": {"base": 500000.0, "dims": 128, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+    gla = {"heads": heads, "dim": 128, "vdim": 128, "tau": 16.0, "decay_rank": 16}
+    dense = {"kind": "dense", "ff": ff}
+    return {"architecture": "Kakirax", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_softcap": 30.0,
+            "embedding": {"scale": 8.0},
+            "layers": [{"type": "attention" if i % 4 == 3 else "gla", "mixer": attn if i % 4 == 3 else gla, "mlp": dense}
+                       for i in range(layers)]}
+
+
 SAKINEX_SIZES = {
     # name: (width, layer runs, heads, experts, top, expert ff, shared ff, window, pool, vocab)
     "small": (2048, 8, 16, 32, 4, 768, 1024, 1024, 64, 32768),
@@ -503,7 +516,8 @@ class _OpTimer:
                  "experts_forward", "attention", "qk_norm_rope_write", "embedding", "logit_post", "attention_prepare",
                  "attention_masked", "convert", "short_conv", "short_conv_state", "min_gru", "scale_rows", "add_scaled",
                  "attention_pooled_prepare", "attention_pool_blocks", "attention_pooled", "zero", "rms_norm_add",
-                 "gate_rows", "gelu_gate", "attention_mixed_heads", "gated_delta", "group_gate_norm"]
+                 "gate_rows", "gelu_gate", "attention_mixed_heads", "gated_delta", "group_gate_norm", "layer_norm",
+                 "gated_linear_attention"]
         for name in names:
             fn = getattr(self.ops, name, None)
             if fn is None:
@@ -588,6 +602,9 @@ def compare_designs(design: str = "sarizen", size: str = "small", steps: int = 6
     elif design == "ziginex":
         width, layers, heads, experts, top, expert_ff, shared_ff, rank, window, vocab = DESIGN_SIZES[size]
         raw = _ziginex_shape(width, layers, heads, experts, top, expert_ff, shared_ff, rank, window, vocab)
+    elif design == "kakirax":
+        width, layers, heads, experts, top, expert_ff, shared_ff, rank, window, vocab = DESIGN_SIZES[size]
+        raw = _kakirax_shape(width, layers, heads, top * expert_ff + shared_ff, vocab)
     else:
         raise ValueError(f"unknown design '{design}'")
     dense = dict(architectures=["Qwen3ForCausalLM"], num_hidden_layers=layers, hidden_size=width,
@@ -604,6 +621,8 @@ def compare_designs(design: str = "sarizen", size: str = "small", steps: int = 6
     others = [("qwen3", dense)]
     if design == "sakinex":     # its closest existing model is the looped design with windows and routed experts
         others.insert(0, ("malapel", _malapel_like_sakinex(width, layers, heads, experts, top, expert_ff, window, vocab)))
+    if design == "kakirax":     # its closest existing model is the hybrid of linear attention with a decaying state and softmax attention
+        others.insert(0, ("sarizen", _sarizen_shape(width, layers, heads, experts, top, expert_ff, shared_ff, rank, window, vocab)))
     if design == "ziginex":     # its closest existing model is the hybrid of a recurrence, latent attention and routed experts
         others.insert(0, ("sarizen", _sarizen_shape(width, layers, heads, experts, top, expert_ff, shared_ff, rank, window, vocab)))
     for name, cfg in [(design, raw)] + others:

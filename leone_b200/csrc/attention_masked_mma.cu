@@ -33,14 +33,6 @@ namespace leone {
 constexpr int kMmRows = 64, kMmKeys = 64, kMmThreads = 128;
 constexpr int kDecKeys = 32;      // keys per tile in the decode form: smaller tiles, more blocks per SM
 
-__device__ __forceinline__ void ldsm4_trans(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
-               : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
-}
-__device__ __forceinline__ uint32_t pack_bf16(float a, float b) {
-  __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
-  return *reinterpret_cast<uint32_t*>(&v);
-}
 // 2^x by the special-function unit (2^-inf = 0); scores are kept in units of log 2 so that a weight
 // costs one subtraction and one of these.
 __device__ __forceinline__ float fast_exp2(float x) {

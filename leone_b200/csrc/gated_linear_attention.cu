@@ -19,66 +19,12 @@
 // Where one block holds all of a head's value columns, it also finishes the head: RMS norm over vdim,
 // weight, times act(gate), stored in the run dtype.
 #include "common.cuh"
+#include "gla_parts.cuh"
 
 namespace leone {
 
 constexpr int kGlaTokens = 16;
 constexpr int kGlaLanes = 32;
-
-// sigmoid(z)^(1/tau) = exp(-softplus(-z) / tau)
-__device__ __forceinline__ float channel_decay(float z, float inv_tau) {
-  const float sp = z < -20.f ? -z : log1pf(expf(-z));
-  return expf(-sp * inv_tau);
-}
-
-struct GlaParams {
-  const float* proj;           // [n_tokens, ld]
-  int ld, q_off, k_off, v_off, u_off;
-  const float* w2;             // [rank, heads * dim]: W_2 transposed
-  const float* w2_bias;        // [heads * dim]
-  int rank;
-  float inv_tau, q_scale;
-  float* state;                // [n_slots, heads, dim, vdim]
-  const int* q_start;
-  const int* slot_ids;
-  int heads, dim, vdim, chunk, n_seqs, n_slots;
-  float* chunk_state;          // [chunks, heads, dim, vdim]
-  float* chunk_decay;          // [chunks, heads, dim]
-  float* out;                  // fp32 [n_tokens, ldo], or null with `gated`
-  int ldo;
-  void* gated;                 // run dtype [n_tokens, ldg]: the finished heads
-  int ldg;
-  const float* norm_w;         // [vdim]
-  int gate_off, gate_act;      // columns of proj; 0 sigmoid, 1 silu
-  float eps;
-  int* status;
-};
-
-// The (sequence, chunk) pair a block works on, its token range and the index of the sequence's chunks.
-struct GlaSpan { int seq, t0, t1, last; };
-
-__device__ __forceinline__ bool gla_span(const GlaParams& p, int z, GlaSpan& sp) {
-  if (p.chunk <= 0) {
-    sp.seq = z;
-    sp.t0 = p.q_start[z];
-    sp.t1 = p.q_start[z + 1];
-    sp.last = 1;
-    return sp.t0 < sp.t1;
-  }
-  for (int b = 0; b < p.n_seqs; ++b) {
-    const int first = p.q_start[b], end = p.q_start[b + 1];
-    const int nc = (end - first + p.chunk - 1) / p.chunk;
-    if (z < nc) {
-      sp.seq = b;
-      sp.t0 = first + z * p.chunk;
-      sp.t1 = min(end, sp.t0 + p.chunk);
-      sp.last = sp.t1 == end;
-      return true;
-    }
-    z -= nc;
-  }
-  return false;
-}
 
 // OUT: outputs written, the walk starts from the chunk's (or the slot's) state; else the chunk's own
 // contribution from a zero state.  T: dtype of the finished heads.
@@ -266,14 +212,17 @@ gla_walk_kernel(const GlaParams p) {
 }
 
 // The pass over a sequence's chunks: entry c of chunk_state holds chunk c's own contribution on entry and
-// the state at chunk c's start on exit.  One thread per state element walks the chunks in order.
-__global__ void __launch_bounds__(256)
+// the state at chunk c's start on exit.  One thread per V state elements (V value columns of one row) walks
+// the chunks in order, eight of them requested at a time.
+template <int V>
+__global__ void __launch_bounds__(128)
 gla_prefix_kernel(const GlaParams p) {
   pdl_trigger();
   pdl_wait();
+  constexpr int kAhead = 8;
   const int s = blockIdx.y;
   const size_t per_seq = (size_t)p.heads * p.dim * p.vdim;
-  const size_t e = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  const size_t e = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * V;
   if (e >= per_seq) return;
   const int slot = p.slot_ids[s];
   if (slot < 0 || slot >= p.n_slots) return;
@@ -282,17 +231,42 @@ gla_prefix_kernel(const GlaParams p) {
   const int nc = (p.q_start[s + 1] - p.q_start[s] + p.chunk - 1) / p.chunk;
   const size_t row = e / p.vdim;                   // head * dim + channel
   const size_t rows = (size_t)p.heads * p.dim;
-  float run = p.state[(size_t)slot * per_seq + e];
-  float carry = 0.f, factor = 1.f;
-  for (int c = 0; c < nc; ++c) {
-    float* at = p.chunk_state + (size_t)(first + c) * per_seq + e;
-    const bool more = c + 1 < nc;
-    const float own = more ? *at : 0.f, f = more ? p.chunk_decay[(size_t)(first + c) * rows + row] : 1.f;
-    if (c > 0) run = fmaf(factor, run, carry);
-    *at = run;
-    carry = own;
-    factor = f;
+  float run[V];
+  const float* at0 = p.state + (size_t)slot * per_seq + e;
+#pragma unroll
+  for (int v = 0; v < V; ++v) run[v] = at0[v];
+  for (int c0 = 0; c0 < nc; c0 += kAhead) {
+    float own[kAhead][V], f[kAhead];
+#pragma unroll
+    for (int i = 0; i < kAhead; ++i) {             // (the last chunk's contribution is not there)
+      const bool more = c0 + i + 1 < nc;
+      const float* at = p.chunk_state + (size_t)(first + c0 + i) * per_seq + e;
+      f[i] = more ? p.chunk_decay[(size_t)(first + c0 + i) * rows + row] : 0.f;
+      if (V == 4) {
+        const float4 x = more ? *reinterpret_cast<const float4*>(at) : make_float4(0.f, 0.f, 0.f, 0.f);
+        own[i][0] = x.x; own[i][1 % V] = x.y; own[i][2 % V] = x.z; own[i][3 % V] = x.w;
+      } else {
+        own[i][0] = more ? at[0] : 0.f;
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < kAhead; ++i) {
+      if (c0 + i < nc) {
+        float* at = p.chunk_state + (size_t)(first + c0 + i) * per_seq + e;
+        if (V == 4) *reinterpret_cast<float4*>(at) = make_float4(run[0], run[1 % V], run[2 % V], run[3 % V]);
+        else at[0] = run[0];
+#pragma unroll
+        for (int v = 0; v < V; ++v) run[v] = fmaf(f[i], run[v], own[i][v]);
+      }
+    }
   }
+}
+
+int launch_gla_prefix(const GlaParams& p, cudaStream_t stream) {
+  const size_t per_seq = (size_t)p.heads * p.dim * p.vdim;
+  if (p.vdim % 4 == 0)
+    return launch_kernel(gla_prefix_kernel<4>, dim3((unsigned)((per_seq / 4 + 127) / 128), p.n_seqs), dim3(128), 0, stream, p);
+  return launch_kernel(gla_prefix_kernel<1>, dim3((unsigned)((per_seq + 127) / 128), p.n_seqs), dim3(128), 0, stream, p);
 }
 
 }  // namespace leone
@@ -358,8 +332,7 @@ extern "C" int leone_gla(int dtype, const float* proj, int ld, int q_off, int k_
   if (chunk > 0) {
     WALK_D(float, grid_z, false);
     if (code != 0) return code;
-    const size_t per_seq = (size_t)heads * dim * vdim;
-    code = launch_kernel(gla_prefix_kernel, dim3((unsigned)((per_seq + 255) / 256), n_seqs), dim3(256), 0, stream, p);
+    code = launch_gla_prefix(p, stream);
     if (code != 0) return code;
   }
   if (dtype == 0) WALK_D(float, grid_z, true);

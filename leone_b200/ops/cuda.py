@@ -583,10 +583,28 @@ class CudaOps:
         # a head wider than a block's columns is normed and gated by a kernel of its own
         whole = vdim <= (128 if dim <= 128 else 64 if dim <= 256 else 32)
         o = None if whole else self._scratch("gla_out", n, hv, torch.float32)
+        gated_arg = _ptr(gated) if whole else c_void_p(0)
+        offsets = (q_off, k_off, v_off, u_off, gate_off)
+        if (self.fast is not None and gated.dtype == torch.bfloat16 and not ctx.decode_only and ctx.max_q_len >= 16
+                and os.environ.get("LEONE_NO_GLA_MMA", "0") != "1" and chunk % 16 == 0 and rank <= 512
+                and self.mixers.leone_gla_mma_supported(dim, vdim)
+                and proj.stride(0) % 4 == 0 and gated.stride(0) % 4 == 0 and not any(o_ % 4 for o_ in offsets if o_ != u_off)):
+            # prompt portions in bfloat16: 16 tokens at a time on tensor cores
+            alpha = self._scratch("gla_alpha", n, heads * dim, torch.float32)
+            self.launches += 2 if chunk == 0 else 4
+            _check(self.mixers.leone_gla_mma(
+                _ptr(proj), proj.stride(0), *offsets, _ptr(w2), _ptr(w2_bias), rank, c_float(1.0 / tau), c_float(q_scale),
+                _ptr(o), 0 if o is None else o.stride(0), gated_arg, gated.stride(0), _ptr(norm_w),
+                1 if act == "silu" else 0, c_float(eps), _ptr(state), _ptr(ctx.q_start), _ptr(ctx.slot_ids), n, ctx.n_seqs,
+                heads, dim, vdim, state.shape[0], chunk, n_chunks, _ptr(chunk_state), _ptr(chunk_decay), _ptr(alpha),
+                _ptr(ctx.status), self._stream()), "gated_linear_attention (tensor cores)")
+            if not whole:
+                self.group_gate_norm(o, norm_w, proj[:, gate_off:gate_off + hv], gated, eps, heads, vdim, act=act)
+            return
         self.launches += 1 if chunk == 0 else 3
         _check(self.mixers.leone_gla(
             _dt(gated.dtype), _ptr(proj), proj.stride(0), q_off, k_off, v_off, u_off, gate_off, _ptr(w2), _ptr(w2_bias), rank,
-            c_float(1.0 / tau), c_float(q_scale), _ptr(o), 0 if o is None else o.stride(0), _ptr(gated) if whole else c_void_p(0),
+            c_float(1.0 / tau), c_float(q_scale), _ptr(o), 0 if o is None else o.stride(0), gated_arg,
             gated.stride(0), _ptr(norm_w), 1 if act == "silu" else 0, c_float(eps), _ptr(state), _ptr(ctx.q_start),
             _ptr(ctx.slot_ids), ctx.n_seqs, heads, dim, vdim, state.shape[0], chunk, n_chunks, _ptr(chunk_state),
             _ptr(chunk_decay), _ptr(ctx.status), self._stream()), "gated_linear_attention")

@@ -70,7 +70,7 @@ class GatedLinearAttention(Mixer):
 
     def scratch_bytes(self, max_tokens):
         chunks = max_tokens // max(self.chunk, 1) + 1
-        return max_tokens * (self.cols * 4 + self.hv * (4 + self.rt.dtype.itemsize)) \
+        return max_tokens * ((self.cols + self.qk) * 4 + self.hv * (4 + self.rt.dtype.itemsize)) \
             + chunks * self.heads * self.dim * (self.vdim + 1) * 4
 
     def load_transient_bytes(self):
