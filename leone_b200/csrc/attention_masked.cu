@@ -128,6 +128,112 @@ attention_prepare_kernel(T* __restrict__ qkv, int row_stride, int n_q, int n_kv,
   }
 }
 
+// The same for bfloat16 heads of DK = 64 or 128 elements with a half-split rotation of all of them (or none) and a
+// norm per head (or none): a warp takes whole heads, a lane E = DK / 32 neighbouring elements, whose rotation
+// partners are the lane 16 away's; no shared memory but the token's cos and sin.
+template <int DK>
+__global__ void __launch_bounds__(kPrepThreads)
+attention_prepare_heads_kernel(__nv_bfloat16* __restrict__ qkv, int row_stride, int n_q, int n_kv, int dv, int norm,
+                               const float* __restrict__ q_w, const float* __restrict__ k_w, float eps,
+                               const float* __restrict__ freqs, const int* __restrict__ positions,
+                               const int* __restrict__ seq_of_token, const int* __restrict__ block_table,
+                               int table_width, int n_seqs, __nv_bfloat16* __restrict__ k_pool,
+                               __nv_bfloat16* __restrict__ v_pool, int num_pages, int page_tokens, int* status) {
+  pdl_trigger();
+  pdl_wait();
+  constexpr int E = DK / 32, HALF = DK / 2;
+  __shared__ float2 cs[HALF];
+  const int t = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, warps = kPrepThreads / 32;
+  const int heads = n_q + n_kv;
+  __nv_bfloat16* row = qkv + (size_t)t * row_stride;
+  const int pos = positions[t];
+  if (pos < 0) {
+    if (tid == 0) set_status(status, kBadPosition, t, pos);
+    return;
+  }
+  if (freqs != nullptr) {
+    for (int i = tid; i < HALF; i += kPrepThreads) {
+      float s, c;
+      sincosf((float)pos * freqs[i], &s, &c);
+      cs[i] = make_float2(c, s);
+    }
+  }
+  long long slot = -1;
+  if (k_pool != nullptr) {
+    const int s = seq_of_token[t];
+    if (s < 0 || s >= n_seqs) {
+      if (tid == 0) set_status(status, kBadSequence, t, s);
+      return;
+    }
+    const int blk = pos / page_tokens;
+    const int page = blk < table_width ? block_table[(size_t)s * table_width + blk] : -1;
+    if (page < 0 || page >= num_pages) {
+      if (tid == 0) set_status(status, kBadPage, t, page, pos);
+      return;
+    }
+    slot = (long long)page * n_kv * page_tokens + (pos % page_tokens);
+  }
+  __syncthreads();
+  for (int h = warp; h < heads; h += warps) {
+    uint32_t raw[E / 2];
+    uint32_t* at = reinterpret_cast<uint32_t*>(row + h * DK) + lane * (E / 2);
+    if (E == 4) {
+      const uint2 r = *reinterpret_cast<const uint2*>(at);
+      raw[0] = r.x;
+      raw[E / 2 - 1] = r.y;
+    } else {
+      raw[0] = at[0];
+    }
+    float x[E];
+#pragma unroll
+    for (int i = 0; i < E / 2; ++i) {
+      x[2 * i] = __uint_as_float(raw[i] << 16);
+      x[2 * i + 1] = __uint_as_float(raw[i] & 0xffff0000u);
+    }
+    if (norm) {
+      float ss = 0.f;
+#pragma unroll
+      for (int i = 0; i < E; ++i) ss = fmaf(x[i], x[i], ss);
+      const float r = 1.f / sqrtf(warp_sum(ss) / (float)DK + eps);
+      const float* w = h < n_q ? q_w : k_w;
+#pragma unroll
+      for (int i = 0; i < E; ++i) x[i] = x[i] * r * w[lane * E + i];
+    }
+    if (freqs != nullptr) {
+#pragma unroll
+      for (int i = 0; i < E; ++i) {
+        const float other = __shfl_xor_sync(0xffffffffu, x[i], 16);
+        const float2 a = cs[(lane & 15) * E + i];
+        x[i] = lane < 16 ? x[i] * a.x - other * a.y : x[i] * a.x + other * a.y;
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < E / 2; ++i) {
+      const __nv_bfloat162 b = __floats2bfloat162_rn(x[2 * i], x[2 * i + 1]);
+      raw[i] = *reinterpret_cast<const uint32_t*>(&b);
+    }
+    uint32_t* page_row = h >= n_q && slot >= 0
+        ? reinterpret_cast<uint32_t*>(k_pool + (slot + (long long)(h - n_q) * page_tokens) * DK) + lane * (E / 2) : nullptr;
+    if (E == 4) {
+      const uint2 r = make_uint2(raw[0], raw[E / 2 - 1]);
+      *reinterpret_cast<uint2*>(at) = r;
+      if (page_row != nullptr) *reinterpret_cast<uint2*>(page_row) = r;
+    } else {
+      at[0] = raw[0];
+      if (page_row != nullptr) page_row[0] = raw[0];
+    }
+  }
+  if (slot >= 0) {
+    const __nv_bfloat16* vrow = row + heads * DK;
+    const int v8 = dv / 8;
+    for (int c = tid; c < n_kv * v8; c += kPrepThreads) {
+      const int h = c / v8, e = (c - h * v8) * 8;
+      *reinterpret_cast<uint4*>(v_pool + (slot + (long long)h * page_tokens) * dv + e) =
+          *reinterpret_cast<const uint4*>(vrow + h * dv + e);
+    }
+  }
+}
+
 constexpr int kMaskedThreads = 128;
 constexpr int kMaskedAcc = 8;          // value width <= 1024
 
@@ -254,6 +360,18 @@ extern "C" int leone_attention_prepare(int dtype, void* qkv, int row_stride, int
   if (rot_dims < 0 || rot_dims > dk || (rot_dims & 1)) return kRefusedSize;
   if (k_pool != nullptr && (v_pool == nullptr || page_tokens <= 0 || table_width <= 0)) return kRefusedSize;
   if (row_stride < (n_q + n_kv) * dk + n_kv * dv) return kRefusedSize;
+  // heads that warps can take whole
+  if (dtype == 1 && (dk == 64 || dk == 128) && dv % 8 == 0 && norm_mode != 2 && !adjacent && (rot_dims == 0 || rot_dims == dk) &&
+      row_stride % 8 == 0 && (((uintptr_t)qkv | (uintptr_t)k_pool | (uintptr_t)v_pool) & 15) == 0) {
+#define HEADS(DK)                                                                                                      \
+  return launch_kernel(attention_prepare_heads_kernel<DK>, dim3(n_tokens), dim3(kPrepThreads), 0, stream,              \
+                       (__nv_bfloat16*)qkv, row_stride, n_q, n_kv, dv, norm_mode, q_w, k_w, eps, rot_dims ? freqs : nullptr, \
+                       positions, seq_of_token, block_table, table_width, n_seqs, (__nv_bfloat16*)k_pool,              \
+                       (__nv_bfloat16*)v_pool, num_pages, page_tokens, status)
+    if (dk == 64) HEADS(64);
+    HEADS(128);
+#undef HEADS
+  }
   const size_t smem = ((size_t)(n_q + n_kv) * dk + (n_q + n_kv) + rot_dims + 2) * sizeof(float);
   if (smem > 200 * 1024) return kRefusedSize;
 #define LAUNCH(T)                                                                                              \

@@ -105,6 +105,7 @@ gla_walk_kernel(const GlaParams p) {
 #pragma unroll
       for (int j = 0; j < 8; ++j) z[j] = b;
       const float* wr = p.w2 + (size_t)h * dim + c;
+#pragma unroll 16
       for (int r = 0; r < p.rank; ++r) {
         const float w = wr[(size_t)r * hd];
         const float4 ua = *reinterpret_cast<const float4*>(u_s + r * kGlaTokens + g * 8);

@@ -38,8 +38,25 @@ __device__ __forceinline__ void split_pair(float a, float b, uint32_t& hi, uint3
   lo = pack_bf16(a - __uint_as_float(hi << 16), b - __uint_as_float(hi & 0xffff0000u));
 }
 
-// alpha[t, c] for 16 tokens a block.  The fast exponential and logarithm are a few units in the last place
-// of fp32 off; near alpha = 1 the logarithm's argument is 1 + small, whose rounding is 6e-8 absolute.
+__device__ __forceinline__ float exp2_fast(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float log2_fast(float x) {
+  float y;
+  asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float rcp_fast(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+// alpha[t, c] = sigmoid(z)^(1/tau) = 2^(-log2(1 + 2^(-z log2 e)) / tau) for 16 tokens a block.  The hardware's powers
+// and logarithms of two are a few units in the last place of fp32 off; near alpha = 1 the logarithm's argument is
+// 1 + small, whose rounding is 6e-8 absolute.
 __global__ void __launch_bounds__(256)
 gla_decay_kernel(const GlaParams p, float* __restrict__ alpha, int n_tokens) {
   pdl_trigger();
@@ -57,6 +74,7 @@ gla_decay_kernel(const GlaParams p, float* __restrict__ alpha, int n_tokens) {
   const float b = p.w2_bias[c];
 #pragma unroll
   for (int j = 0; j < kGmTokens; ++j) z[j] = b;
+#pragma unroll 8
   for (int r = 0; r < p.rank; ++r) {
     const float w = p.w2[(size_t)r * hd + c];
 #pragma unroll
@@ -68,12 +86,13 @@ gla_decay_kernel(const GlaParams p, float* __restrict__ alpha, int n_tokens) {
       z[j + 3] = fmaf(w, u.w, z[j + 3]);
     }
   }
+  float* dst = alpha + (size_t)tb * hd + c;
 #pragma unroll
-  for (int j = 0; j < kGmTokens; ++j)
-    if (j < nt) {
-      const float sp = z[j] < -20.f ? -z[j] : __logf(1.f + __expf(-z[j]));
-      alpha[(size_t)(tb + j) * hd + c] = __expf(-sp * p.inv_tau);
-    }
+  for (int j = 0; j < kGmTokens; ++j) {
+    const float y = -1.4426950408889634f * z[j];
+    const float sp = y > 30.f ? y : log2_fast(1.f + exp2_fast(y));      // softplus(-z) in units of log 2
+    if (j < nt) dst[(size_t)j * hd] = exp2_fast(-sp * p.inv_tau);
+  }
 }
 
 template <int KD> struct GmLayout {
@@ -172,7 +191,7 @@ gla_mma_kernel(const GlaParams p, const float* __restrict__ alpha) {
     {
       const int job = tid >> 6, c = (tid & 63) * 2;
       if (job == 3) {
-#pragma unroll 4
+#pragma unroll 2
         for (int tt = 0; tt < kGmTokens; ++tt) {
           const float2 x = *reinterpret_cast<const float2*>(v_s + tt * kGmCols + c);
           uint32_t hi, lo;
@@ -184,7 +203,7 @@ gla_mma_kernel(const GlaParams p, const float* __restrict__ alpha) {
         const bool in0 = c < dim, in1 = c + 1 < dim;
         float p0 = 1.f, p1 = 1.f;
         if (job == 2) {                            // from the last token back
-#pragma unroll 4
+#pragma unroll 2
           for (int tt = kGmTokens - 1; tt >= 0; --tt) {
             const float2 k = *reinterpret_cast<const float2*>(k_s + tt * DIMP + c);
             uint32_t hi, lo;
@@ -205,7 +224,7 @@ gla_mma_kernel(const GlaParams p, const float* __restrict__ alpha) {
         } else {
           const float* src = job == 0 ? q_s : k_s;
           __nv_bfloat16* dst = job == 0 ? qh : ih;
-#pragma unroll 4
+#pragma unroll 2
           for (int tt = 0; tt < kGmTokens; ++tt) {
             if (tt < nt) {
               const float2 a = *reinterpret_cast<const float2*>(a_s + tt * DIMP + c);
@@ -213,7 +232,7 @@ gla_mma_kernel(const GlaParams p, const float* __restrict__ alpha) {
               if (in1) p1 *= a.y;
             }
             const float2 x = *reinterpret_cast<const float2*>(src + tt * DIMP + c);
-            const float f0 = job == 0 ? p0 * p.q_scale : __fdividef(1.f, p0), f1 = job == 0 ? p1 * p.q_scale : __fdividef(1.f, p1);
+            const float f0 = job == 0 ? p0 * p.q_scale : rcp_fast(p0), f1 = job == 0 ? p1 * p.q_scale : rcp_fast(p1);
             uint32_t hi, lo;
             split_pair(x.x * f0, x.y * f1, hi, lo);
             *reinterpret_cast<uint32_t*>(dst + tt * PD + c) = hi;

@@ -212,6 +212,30 @@ gate_rows_kernel(T* __restrict__ a, int lda, const T* __restrict__ gate, int ldg
   }
 }
 
+// The same with eight bfloat16 columns a thread (rows, columns and bases that 16-byte accesses fit).
+__global__ void __launch_bounds__(256)
+gate_rows_vec_kernel(__nv_bfloat16* __restrict__ a, int lda, const __nv_bfloat16* __restrict__ gate, int ldg, int n_rows,
+                     int cols8, int act) {
+  pdl_trigger();
+  pdl_wait();
+  const int c = blockIdx.x * blockDim.x + threadIdx.x;
+  if (c >= cols8) return;
+  for (int t = blockIdx.y; t < n_rows; t += gridDim.y) {
+    uint4* at = reinterpret_cast<uint4*>(a + (size_t)t * lda) + c;
+    const uint4 zr = *(reinterpret_cast<const uint4*>(gate + (size_t)t * ldg) + c);
+    uint4 ar = *at;
+    const __nv_bfloat162* z2 = reinterpret_cast<const __nv_bfloat162*>(&zr);
+    __nv_bfloat162* a2 = reinterpret_cast<__nv_bfloat162*>(&ar);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float2 z = __bfloat1622float2(z2[i]), x = __bfloat1622float2(a2[i]);
+      const float s0 = 1.f / (1.f + expf(-z.x)), s1 = 1.f / (1.f + expf(-z.y));
+      a2[i] = __floats2bfloat162_rn(x.x * (act == 1 ? z.x * s0 : s0), x.y * (act == 1 ? z.y * s1 : s1));
+    }
+    *at = ar;
+  }
+}
+
 // out[t, c] = gelu_tanh(z[t, c]) * rows[t, off + c]: a projection's fp32 result gates a slice of a
 // per-token row.  gelu_tanh(z) = z/2 (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))).
 template <typename T>
@@ -320,6 +344,11 @@ extern "C" int leone_gate_rows(int dtype, void* a, int lda, const void* gate, in
   if (n_rows <= 0 || cols <= 0) return 0;
   const long long want = ((long long)n_rows * cols + 255) / 256;
   const unsigned blocks = (unsigned)(want < 148 * 16 ? want : 148 * 16);
+  if (dtype == 1 && cols % 8 == 0 && lda % 8 == 0 && ldg % 8 == 0 && (((uintptr_t)a | (uintptr_t)gate) & 15) == 0) {
+    const int c8 = cols / 8, threads = c8 >= 256 ? 256 : (c8 + 31) / 32 * 32;
+    return launch_kernel(gate_rows_vec_kernel, dim3((c8 + threads - 1) / threads, n_rows < 65535 ? n_rows : 65535), dim3(threads),
+                         0, stream, (__nv_bfloat16*)a, lda, (const __nv_bfloat16*)gate, ldg, n_rows, c8, act);
+  }
   if (dtype == 0)
     return launch_kernel(gate_rows_kernel<float>, dim3(blocks), dim3(256), 0, stream, (float*)a, lda, (const float*)gate,
                          ldg, n_rows, cols, act);

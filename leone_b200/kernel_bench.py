@@ -413,6 +413,54 @@ def bench_gated_delta(ops, tokens, batch, heads, kv_heads, dim, vdim, reps, warm
     return row
 
 
+def bench_gla(ops, tokens, batch, heads, dim, vdim, rank, chunk, reps, warmup):
+    """Gated linear attention with a decay per key channel (``CudaOps.gated_linear_attention``, the heads' norm
+    and gate included): one prompt of ``tokens`` tokens, or with ``batch`` a decode step of that many sequences."""
+    decode = batch > 0
+    seqs, q_len = (batch, 1) if decode else (1, tokens)
+    ctx = _step_of(seqs, q_len, q_len)
+    n, hd, hv = ctx.n_tokens, heads * dim, heads * vdim
+    cols = -(-(2 * hd + 2 * hv + rank) // 16) * 16
+    copies = 1 if not decode else max(1, int(300e6 // (seqs * hd * vdim * 4)) + 1)      # states larger together than L2
+    proj = torch.randn((n, cols), device=DEV)
+    out = torch.empty((n, hv), device=DEV, dtype=torch.bfloat16)
+    states = [torch.zeros((seqs, heads, dim, vdim), device=DEV) for _ in range(copies)]
+    w2, bias, norm_w = torch.randn((rank, hd), device=DEV), torch.zeros(hd, device=DEV), torch.ones(vdim, device=DEV)
+    turn = {"i": 0}
+
+    def run():
+        turn["i"] = (turn["i"] + 1) % copies
+        ops.gated_linear_attention(ctx, proj, out, states[turn["i"]], w2, bias, norm_w, heads, dim, vdim, rank, 16.0,
+                                   dim ** -0.5, 1e-6, q_off=0, k_off=hd, v_off=2 * hd, u_off=2 * hd + 2 * hv,
+                                   gate_off=2 * hd + hv, chunk=chunk if q_len > 2 * chunk else 0)
+    ms = _time(run, reps, warmup, per_graph=copies if decode else 1)
+    moved = n * (cols * 4.0 + hv * 2) + 2.0 * seqs * hd * vdim * 4
+    row = dict(kernel="gated_linear_attention", heads=heads, dim=dim, vdim=vdim, us=ms * 1e3, gbs=moved / ms / 1e6,
+               fp32_tflops=4.0 * n * hd * vdim / ms / 1e9)
+    row.update(dict(batch=batch) if decode else dict(tokens=tokens, chunk=chunk))
+    return row
+
+
+def bench_row_kernels(ops, tokens, width, reps, warmup):
+    """Kernels that pass over rows once: the two norms of the fp32 stream, the output gate."""
+    copies = max(1, min(64, int(300e6 // (tokens * width * 4)) + 1))
+    xs = [torch.randn((tokens, width), device=DEV) for _ in range(copies)]
+    rows16 = [torch.randn((tokens, 2 * width), device=DEV).to(torch.bfloat16) for _ in range(copies)]
+    w, b = torch.ones(width, device=DEV).to(torch.bfloat16), torch.zeros(width, device=DEV).to(torch.bfloat16)
+    out = torch.empty((tokens, width), device=DEV, dtype=torch.bfloat16)
+    turn, rows = {"i": 0}, []
+
+    def step(items):
+        turn["i"] = (turn["i"] + 1) % copies
+        return items[turn["i"]]
+    for name, moved, fn in (("rms_norm", 6, lambda: ops.rms_norm(step(xs), w, out, 1e-6)),
+                            ("layer_norm", 6, lambda: ops.layer_norm(step(xs), w, b, out, 1e-6)),
+                            ("gate_rows", 6, lambda: ops.gate_rows(out, step(rows16)[:, width:]))):
+        ms = _time(fn, reps, warmup, per_graph=copies)
+        rows.append(dict(kernel=name, tokens=tokens, width=width, us=ms * 1e3, gbs=moved * tokens * width / ms / 1e6))
+    return rows
+
+
 def bench_sampling(ops, rows, vocab, stages, reps, warmup):
     """The sampler's truncation pipeline (sort, stages, draw) on ``rows`` rows of ``vocab`` logits;
     wall time with a synchronize on both sides (the call makes dozens of small launches)."""
@@ -435,17 +483,19 @@ def bench_sampling(ops, rows, vocab, stages, reps, warmup):
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(prog="python -m leone_b200.kernel_bench")
     ap.add_argument("what", choices=["gemm", "decode-attention", "prefill-attention", "layer-shapes", "sampling",
-                                     "masked-attention", "pooled-attention", "conv-gru", "mixed-attention", "gated-delta"])
+                                     "masked-attention", "pooled-attention", "conv-gru", "mixed-attention", "gated-delta", "gla",
+                                     "row-kernels"])
     ap.add_argument("--pool", type=int, default=64, help="pooled-attention: positions per pooled block")
     ap.add_argument("--taps", type=int, default=4, help="pooled-attention, conv-gru: taps of the short convolutions")
-    ap.add_argument("--width", type=int, default=2048, help="conv-gru: channels")
-    ap.add_argument("--chunk", type=int, default=None, help="conv-gru: tokens per chunk of the recurrence (default: the part's)")
+    ap.add_argument("--width", type=int, default=2048, help="conv-gru: channels; row-kernels: columns")
+    ap.add_argument("--rank", type=int, default=16, help="gla: inner width of the decay's projection")
+    ap.add_argument("--chunk", type=int, default=None, help="conv-gru, gla: tokens per chunk of the recurrence (default: the part's)")
     ap.add_argument("--mask", choices=["causal", "window", "chunk"], default="window")
     ap.add_argument("--mask-size", type=int, default=1024)
     ap.add_argument("--weights", choices=["softmax", "softmax_plus_one", "sigmoid"], default="sigmoid")
     ap.add_argument("--value-dim", type=int, default=0, help="masked-attention: value width (default: the head size)")
     ap.add_argument("--decode", action="store_true",
-                    help="masked-attention, pooled-attention, mixed-attention, gated-delta, conv-gru: a decode step of --batch sequences")
+                    help="masked-attention, pooled-attention, mixed-attention, gated-delta, gla, conv-gru: a decode step of --batch sequences")
     ap.add_argument("--stages", default="top_k=40,top_p=0.95",
                     help="sampling: truncation stages in order, e.g. top_k=40,typical=0.9")
     ap.add_argument("--vocab", type=int, default=151936)
@@ -539,6 +589,11 @@ def main(argv=None) -> int:
     elif args.what == "gated-delta":
         rows.append(bench_gated_delta(CudaOps(DEV, torch.float32), args.tokens, args.batch if args.decode else 0, args.heads,
                                       args.kv_heads, args.head_dim, args.value_dim or args.head_dim, args.reps, args.warmup))
+    elif args.what == "gla":
+        rows.append(bench_gla(ops, args.tokens, args.batch if args.decode else 0, args.heads, args.head_dim,
+                              args.value_dim or args.head_dim, args.rank, args.chunk or 64, args.reps, args.warmup))
+    elif args.what == "row-kernels":
+        rows += bench_row_kernels(ops, args.tokens, args.width, args.reps, args.warmup)
     elif args.what == "conv-gru":
         from .parts.min_gru import DEFAULT_CHUNK
         rows += bench_conv_and_gru(ops, args.tokens, args.batch if args.decode else 0, args.width, args.taps,

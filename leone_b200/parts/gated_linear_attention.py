@@ -34,8 +34,8 @@ class GatedLinearAttention(Mixer):
         self.q_scale = float(params.get("q_scale", self.dim ** -0.5))
         self.names = {k: params.get(f"{k}_name", k) for k in ("q", "k", "v", "g", "a1", "a2", "o", "norm")}
         self.names["a2_bias"] = params.get("a2_bias_name", f"{self.names['a2']}.b")
-        # prompt portions longer than twice this are cut into chunks that run side by side
-        self.chunk = int(params.get("chunk", 64))
+        # tokens per chunk of a long prompt portion (the chunks run side by side); None: from the step's size
+        self.fixed_chunk = int(params["chunk"]) if params.get("chunk") else None
         self.qk = self.heads * self.dim
         self.hv = self.heads * self.vdim
         # rows of the one input product: q, k, v, the gate, the decay's low-rank part
@@ -69,7 +69,7 @@ class GatedLinearAttention(Mixer):
         return (self.cols * self.hidden + self.hidden * self.hv) * self.rt.dtype.itemsize + self.rank * self.qk * 4
 
     def scratch_bytes(self, max_tokens):
-        chunks = max_tokens // max(self.chunk, 1) + 1
+        chunks = max_tokens // self.chunk_for(max_tokens) + 1
         return max_tokens * ((self.cols + self.qk) * 4 + self.hv * (4 + self.rt.dtype.itemsize)) \
             + chunks * self.heads * self.dim * (self.vdim + 1) * 4
 
@@ -79,13 +79,23 @@ class GatedLinearAttention(Mixer):
     def cache_request(self):
         return FixedState((self.heads, self.dim, self.vdim))
 
+    def chunk_for(self, tokens):
+        """The longest chunk (a power of two from 32 to 256) that leaves about a block and a half for each of
+        148 SMs: longer chunks move fewer states between the kernels, but an SM without a block does nothing."""
+        chunk = self.fixed_chunk or 32
+        while self.fixed_chunk is None and chunk < 256 and tokens * self.heads >= 2 * chunk * 200:
+            chunk *= 2
+        return chunk
+
     def forward(self, ctx, cache, x, hidden, fresh=False):
         rt, ops = self.rt, self.rt.ops
         n = hidden.shape[0]
         proj = rt.buffer("gla_proj", n, self.cols, torch.float32)
         ops.linear(x, self.w_in, proj)
         # a captured step has one token per sequence; otherwise long portions run chunk-parallel
-        chunk = self.chunk if not ctx.decode_only and self.chunk > 0 and ctx.max_q_len > 2 * self.chunk else 0
+        chunk = 0 if ctx.decode_only else self.chunk_for(n)
+        if ctx.max_q_len <= 2 * chunk:
+            chunk = 0
         gated = rt.buffer("gla_gated", n, self.hv, rt.dtype)
         ops.gated_linear_attention(ctx, proj, gated, cache.state, self.w2, self.w2_bias, self.norm_w, self.heads, self.dim,
                                    self.vdim, self.rank, self.tau, self.q_scale, self.eps, q_off=0, k_off=self.qk,
