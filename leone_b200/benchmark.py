@@ -483,6 +483,23 @@ def _kakirax_shape(width: int, layers: int, heads: int, ff: int, vocab: int) -> 
                        for i in range(layers)]}
 
 
+def _gulipel_shape(width: int, layers: int, heads: int, ff: int, vocab: int) -> dict:
+    """Layer sizes that resemble a real model's: three Mamba-2 layers (inner width twice the model's, heads of 64, a
+    state of 128, eight groups of B and C) to every parallel layer (attention with four query heads to a key/value head
+    beside a delta rule with a decay per key channel, inner widths of 128, convolutions of four taps); a dense
+    feed-forward and a token gate of 256 everywhere; pairs of tokens in 65,521 rows."""
+    mamba = {"heads": 2 * width // 64, "vdim": 64, "state": 128, "groups": 8, "norm_groups": 8, "conv": 4}
+    left = {"heads": heads, "kv_heads": max(heads // 4, 1), "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+            "q_temp": {"coef": 0.1, "every": 8192}}
+    right = {"heads": heads, "kv_heads": heads, "dim": 128, "vdim": 128, "conv": 4, "decay_rank": 128, "gate_rank": 128}
+    dense = {"kind": "dense", "ff": ff}
+    return {"architecture": "Gulipel", "vocab": vocab, "width": width, "max_positions": 16384, "norm": {"eps": 1e-6},
+            "embedding": {"scale": 8.0, "bigram": {"buckets": 65521, "mul_prev": 31, "mul_cur": 17}},
+            "token_side": {"dim": 256}, "logit_softcap": 30.0,
+            "layers": [{"type": "parallel", "mixer": {"left": left, "right": right}, "mlp": dense} if i % 4 == 3 else
+                       {"type": "mamba2", "mixer": mamba, "mlp": dense} for i in range(layers)]}
+
+
 SAKINEX_SIZES = {
     # name: (width, layer runs, heads, experts, top, expert ff, shared ff, window, pool, vocab)
     "small": (2048, 8, 16, 32, 4, 768, 1024, 1024, 64, 32768),
@@ -517,7 +534,7 @@ class _OpTimer:
                  "attention_masked", "convert", "short_conv", "short_conv_state", "min_gru", "scale_rows", "add_scaled",
                  "attention_pooled_prepare", "attention_pool_blocks", "attention_pooled", "zero", "rms_norm_add",
                  "gate_rows", "gelu_gate", "attention_mixed_heads", "gated_delta", "group_gate_norm", "layer_norm",
-                 "gated_linear_attention"]
+                 "gated_linear_attention", "embedding_sum", "ssd", "grouped_gate_norm"]
         for name in names:
             fn = getattr(self.ops, name, None)
             if fn is None:
@@ -605,6 +622,9 @@ def compare_designs(design: str = "sarizen", size: str = "small", steps: int = 6
     elif design == "kakirax":
         width, layers, heads, experts, top, expert_ff, shared_ff, rank, window, vocab = DESIGN_SIZES[size]
         raw = _kakirax_shape(width, layers, heads, top * expert_ff + shared_ff, vocab)
+    elif design == "gulipel":
+        width, layers, heads, experts, top, expert_ff, shared_ff, rank, window, vocab = DESIGN_SIZES[size]
+        raw = _gulipel_shape(width, layers, heads, top * expert_ff + shared_ff, vocab)
     else:
         raise ValueError(f"unknown design '{design}'")
     dense = dict(architectures=["Qwen3ForCausalLM"], num_hidden_layers=layers, hidden_size=width,
@@ -623,6 +643,9 @@ def compare_designs(design: str = "sarizen", size: str = "small", steps: int = 6
         others.insert(0, ("malapel", _malapel_like_sakinex(width, layers, heads, experts, top, expert_ff, window, vocab)))
     if design == "kakirax":     # its closest existing model is the hybrid of linear attention with a decaying state and softmax attention
         others.insert(0, ("sarizen", _sarizen_shape(width, layers, heads, experts, top, expert_ff, shared_ff, rank, window, vocab)))
+    if design == "gulipel":     # its closest relatives: the other delta rule beside attention, and the other chunked recurrence
+        others.insert(0, ("kakirax", _kakirax_shape(width, layers, heads, top * expert_ff + shared_ff, vocab)))
+        others.insert(0, ("ziginex", _ziginex_shape(width, layers, heads, experts, top, expert_ff, shared_ff, rank, window, vocab)))
     if design == "ziginex":     # its closest existing model is the hybrid of a recurrence, latent attention and routed experts
         others.insert(0, ("sarizen", _sarizen_shape(width, layers, heads, experts, top, expert_ff, shared_ff, rank, window, vocab)))
     for name, cfg in [(design, raw)] + others:

@@ -13,7 +13,8 @@
 // heads at once with weights [n_q dk] and [n_kv dk]; the weight multiplies directly), then the
 // rotation of the first rot_dims elements of every q and k head by position * freq[pair] (pair i is
 // elements (i, i + rot_dims/2), or (2i, 2i + 1) with `adjacent`; angle, cos and sin formed in fp32),
-// q and k written back in place, k into the key page and v into the value page of the token.
+// q and k written back in place, k into the key page and v into the value page of the token.  temp_every > 0: q is
+// multiplied by 1 + temp_coef * ln(floor((position + 1) / temp_every) + 1) on the way, in fp32.
 //
 // leone_attention_masked: one block per (token, query head); scores and weights in fp32, online
 // over tiles of 128 keys in ascending order.  The softmax with the silent member is the ordinary
@@ -25,11 +26,16 @@ namespace leone {
 
 constexpr int kPrepThreads = 256;
 
+// The factor on a query at position pos (1 without a temperature).
+__device__ __forceinline__ float query_temperature(int pos, float coef, int every) {
+  return every > 0 ? 1.f + coef * logf((float)((pos + 1) / every + 1)) : 1.f;
+}
+
 template <typename T>
 __global__ void __launch_bounds__(kPrepThreads)
 attention_prepare_kernel(T* __restrict__ qkv, int row_stride, int n_q, int n_kv, int dk, int dv, int norm_mode,
                          const float* __restrict__ q_w, const float* __restrict__ k_w, float eps,
-                         const float* __restrict__ freqs, int rot_dims, int adjacent,
+                         const float* __restrict__ freqs, int rot_dims, int adjacent, float temp_coef, int temp_every,
                          const int* __restrict__ positions, const int* __restrict__ seq_of_token,
                          const int* __restrict__ block_table, int table_width, int n_seqs,
                          T* __restrict__ k_pool, T* __restrict__ v_pool, int num_pages, int page_tokens,
@@ -105,6 +111,7 @@ attention_prepare_kernel(T* __restrict__ qkv, int row_stride, int n_q, int n_kv,
     key_at = slot * dk;          // kv head h adds h * page_tokens * dk
     value_at = slot * dv;
   }
+  const float temp = query_temperature(pos, temp_coef, temp_every);
   for (int c = tid; c < qk; c += kPrepThreads) {
     const int h = c / dk, e = c - h * dk;
     float v = buf[c];
@@ -115,6 +122,7 @@ attention_prepare_kernel(T* __restrict__ qkv, int row_stride, int n_q, int n_kv,
       const float co = cs[2 * pair], si = cs[2 * pair + 1];
       v = first ? a * co - b * si : b * co + a * si;
     }
+    if (h < n_q) v *= temp;
     const T o = from_float<T>(v);
     row[c] = o;
     if (h >= n_q && key_at >= 0) k_pool[key_at + (long long)(h - n_q) * page_tokens * dk + e] = o;
@@ -135,8 +143,8 @@ template <int DK>
 __global__ void __launch_bounds__(kPrepThreads)
 attention_prepare_heads_kernel(__nv_bfloat16* __restrict__ qkv, int row_stride, int n_q, int n_kv, int dv, int norm,
                                const float* __restrict__ q_w, const float* __restrict__ k_w, float eps,
-                               const float* __restrict__ freqs, const int* __restrict__ positions,
-                               const int* __restrict__ seq_of_token, const int* __restrict__ block_table,
+                               const float* __restrict__ freqs, float temp_coef, int temp_every,
+                               const int* __restrict__ positions, const int* __restrict__ seq_of_token, const int* __restrict__ block_table,
                                int table_width, int n_seqs, __nv_bfloat16* __restrict__ k_pool,
                                __nv_bfloat16* __restrict__ v_pool, int num_pages, int page_tokens, int* status) {
   pdl_trigger();
@@ -173,6 +181,7 @@ attention_prepare_heads_kernel(__nv_bfloat16* __restrict__ qkv, int row_stride, 
     }
     slot = (long long)page * n_kv * page_tokens + (pos % page_tokens);
   }
+  const float temp = query_temperature(pos, temp_coef, temp_every);
   __syncthreads();
   for (int h = warp; h < heads; h += warps) {
     uint32_t raw[E / 2];
@@ -206,6 +215,10 @@ attention_prepare_heads_kernel(__nv_bfloat16* __restrict__ qkv, int row_stride, 
         const float2 a = cs[(lane & 15) * E + i];
         x[i] = lane < 16 ? x[i] * a.x - other * a.y : x[i] * a.x + other * a.y;
       }
+    }
+    if (h < n_q) {
+#pragma unroll
+      for (int i = 0; i < E; ++i) x[i] *= temp;
     }
 #pragma unroll
     for (int i = 0; i < E / 2; ++i) {
@@ -349,13 +362,14 @@ using namespace leone;
 // k_pool null: nothing is written into pages (a layer that reads another layer's cache).
 extern "C" int leone_attention_prepare(int dtype, void* qkv, int row_stride, int n_tokens, int n_q, int n_kv, int dk,
                                        int dv, int norm_mode, const float* q_w, const float* k_w, float eps,
-                                       const float* freqs, int rot_dims, int adjacent, const int* positions,
-                                       const int* seq_of_token, const int* block_table, int table_width, int n_seqs,
+                                       const float* freqs, int rot_dims, int adjacent, float temp_coef, int temp_every,
+                                       const int* positions, const int* seq_of_token, const int* block_table, int table_width, int n_seqs,
                                        void* k_pool, void* v_pool, int num_pages, int page_tokens, int* status,
                                        cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
   if (dk <= 0 || dv <= 0 || n_q <= 0 || n_kv <= 0 || norm_mode < 0 || norm_mode > 2) return kRefusedSize;
   if (norm_mode != 0 && (q_w == nullptr || k_w == nullptr)) return kRefusedSize;
+  if (temp_every < 0) return kRefusedSize;
   if (freqs == nullptr) rot_dims = 0;
   if (rot_dims < 0 || rot_dims > dk || (rot_dims & 1)) return kRefusedSize;
   if (k_pool != nullptr && (v_pool == nullptr || page_tokens <= 0 || table_width <= 0)) return kRefusedSize;
@@ -366,7 +380,7 @@ extern "C" int leone_attention_prepare(int dtype, void* qkv, int row_stride, int
 #define HEADS(DK)                                                                                                      \
   return launch_kernel(attention_prepare_heads_kernel<DK>, dim3(n_tokens), dim3(kPrepThreads), 0, stream,              \
                        (__nv_bfloat16*)qkv, row_stride, n_q, n_kv, dv, norm_mode, q_w, k_w, eps, rot_dims ? freqs : nullptr, \
-                       positions, seq_of_token, block_table, table_width, n_seqs, (__nv_bfloat16*)k_pool,              \
+                       temp_coef, temp_every, positions, seq_of_token, block_table, table_width, n_seqs, (__nv_bfloat16*)k_pool,              \
                        (__nv_bfloat16*)v_pool, num_pages, page_tokens, status)
     if (dk == 64) HEADS(64);
     HEADS(128);
@@ -380,7 +394,7 @@ extern "C" int leone_attention_prepare(int dtype, void* qkv, int row_stride, int
       cudaFuncSetAttribute(attention_prepare_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
     return launch_kernel(attention_prepare_kernel<T>, dim3(n_tokens), dim3(kPrepThreads), smem, stream, (T*)qkv, \
                          row_stride, n_q, n_kv, dk, dv, norm_mode, q_w, k_w, eps, freqs, rot_dims, adjacent,      \
-                         positions, seq_of_token, block_table, table_width, n_seqs, (T*)k_pool, (T*)v_pool,      \
+                         temp_coef, temp_every, positions, seq_of_token, block_table, table_width, n_seqs, (T*)k_pool, (T*)v_pool,      \
                          num_pages, page_tokens, status);                                                        \
   }
   if (dtype == 0) LAUNCH(float);

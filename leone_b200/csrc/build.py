@@ -35,11 +35,11 @@ MODULES: Dict[str, List[str]] = {
     # linear attention with a decaying state, attention through a cached latent, attention with a choice
     # of mask and weight rule, routed experts, short convolutions with state, the minGRU recurrence, attention
     # over a window of tokens and pooled blocks before it, attention whose scores are mixed across heads, the gated
-    # delta rule, gated linear attention with a decay per key channel
+    # delta rule, gated linear attention with a decay per key channel, the Mamba-2 recurrence
     "mixers": ["linear_attention.cu", "attention_latent.cu", "attention_latent_mma.cu", "attention_masked.cu",
                "attention_masked_mma.cu", "experts.cu", "norm_act.cu", "short_conv.cu", "attention_pooled.cu",
                "attention_mixed_heads.cu", "attention_mixed_heads_mma.cu", "gated_delta.cu",
-               "gated_linear_attention.cu", "gated_linear_attention_mma.cu"],
+               "gated_linear_attention.cu", "gated_linear_attention_mma.cu", "ssd.cu"],
     # the entry point that allocates nothing (leone_static.h); it compiles attention_tiled.cu in
     "static": ["attention_decode_static.cu"],
     # the host side of the runtime (pages, block tables, step metadata, the scheduler's decisions,
@@ -48,7 +48,7 @@ MODULES: Dict[str, List[str]] = {
 }
 HOST_ONLY = {"host"}
 HEADERS = ["common.cuh", "mma_tile.cuh", "tc_common.cuh", "gemm_parts.cuh", "leone_static.h", "attention_tiled.cu", "random_draw.h",
-           "gla_parts.cuh"]
+           "gla_parts.cuh", "ssd_parts.cuh"]
 
 # -fno-gnu-unique: statics inside inline functions and templates (the once-per-kernel set-up
 # flags, the launch mode switch) must belong to one library image each; with GNU unique

@@ -641,6 +641,71 @@ __global__ void decode_advance_kernel(int* token_ids, int* positions, int* ctx_l
   if (threadIdx.x == 0) *step_counter = step + 1;
 }
 
+// out[t] = scale * table[id_t] + pairs[row_t] + places[position_t]: a token's row, a row of a second table chosen by
+// the pair (previous token, token), row_t = (previous * mul_prev + id_t * mul_cur) mod buckets, or row `buckets` at a
+// sequence's first position, and a row per position; either of the two may be absent (null).  The previous token of a
+// sequence's first token in the step comes from the sequence's state (one 32-bit word per slot that holds a token id);
+// the block of that token, the only reader of the word, leaves the sequence's last token of the step there.
+template <typename T>
+__global__ void embedding_sum_kernel(const T* __restrict__ table, const int* __restrict__ ids, float* __restrict__ out,
+                                     int hidden, int vocab, float scale, const T* __restrict__ pairs, int buckets,
+                                     long long mul_prev, long long mul_cur, int* last_token, int write_state,
+                                     const T* __restrict__ places, int n_places, const int* __restrict__ positions,
+                                     const int* __restrict__ q_start, const int* __restrict__ seq_of_token,
+                                     const int* __restrict__ slot_ids, int n_seqs, int n_slots, int* status) {
+  pdl_trigger();
+  pdl_wait();
+  const int row = blockIdx.x;
+  const int id = ids[row], pos = positions[row];
+  float* dst = out + (size_t)row * hidden;
+  const T *pair = nullptr, *place = nullptr;
+  bool ok = id >= 0 && id < vocab;
+  if (!ok && threadIdx.x == 0) set_status(status, kBadTokenId, row, id);
+  if (ok && places != nullptr) {
+    ok = pos >= 0 && pos < n_places;
+    if (ok) place = places + (size_t)pos * hidden;
+    else if (threadIdx.x == 0) set_status(status, kBadPosition, row, pos);
+  }
+  int* word = nullptr;
+  int next = 0;
+  if (ok && pairs != nullptr) {
+    const int s = seq_of_token[row];
+    const int slot = s >= 0 && s < n_seqs ? slot_ids[s] : -1;
+    if (slot < 0 || slot >= n_slots) {
+      if (threadIdx.x == 0) set_status(status, kBadSequence, row, s);
+      ok = false;
+    } else {
+      const bool first = row == q_start[s];
+      long long at = buckets;
+      if (pos > 0) {
+        const long long before = first ? last_token[slot] : ids[row - 1];
+        at = (before * mul_prev + (long long)id * mul_cur) % buckets;
+        if (at < 0) at += buckets;
+      }
+      pair = pairs + (size_t)at * hidden;
+      if (first && write_state) {
+        word = last_token + slot;
+        next = ids[q_start[s + 1] - 1];
+      }
+    }
+  }
+  if (!ok) {                                       // (the whole block agrees)
+    for (int c = threadIdx.x; c < hidden; c += blockDim.x) dst[c] = 0.f;
+    return;
+  }
+  const T* src = table + (size_t)id * hidden;
+  for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
+    float v = to_float<T>(src[c]) * scale;
+    if (pair != nullptr) v += to_float<T>(pair[c]);
+    if (place != nullptr) v += to_float<T>(place[c]);
+    dst[c] = v;
+  }
+  if (word != nullptr) {
+    __syncthreads();                               // every thread has read the word
+    if (threadIdx.x == 0) *word = next;
+  }
+}
+
 }  // namespace leone
 
 using namespace leone;
@@ -664,6 +729,28 @@ extern "C" int leone_logit_post(float* logits, long long n, float scale, float c
   const long long want = (n + 255) / 256;
   return launch_kernel(logit_post_kernel, dim3((unsigned)(want < 148 * 8 ? want : 148 * 8)), dim3(256), 0, stream,
                        logits, n, scale, cap);
+}
+
+// pairs: [buckets + 1, hidden] or null (then last_token, q_start, seq_of_token and slot_ids are not read);
+// last_token: int32 [n_slots]; places: [n_places, hidden] or null.
+extern "C" int leone_embedding_sum(int dtype, const void* table, const int* ids, float* out, int n, int hidden, int vocab,
+                                   float scale, const void* pairs, int buckets, long long mul_prev, long long mul_cur,
+                                   int* last_token, int write_state, const void* places, int n_places,
+                                   const int* positions, const int* q_start, const int* seq_of_token,
+                                   const int* slot_ids, int n_seqs, int n_slots, int* status, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (hidden <= 0 || vocab <= 0 || (pairs != nullptr && (buckets <= 0 || last_token == nullptr || n_slots <= 0)) ||
+      (places != nullptr && n_places <= 0))
+    return kRefusedSize;
+  const int threads = hidden >= 1024 ? 256 : 128;
+#define SUM(T)                                                                                                          \
+  return launch_kernel(embedding_sum_kernel<T>, dim3(n), dim3(threads), 0, stream, (const T*)table, ids, out, hidden,   \
+                       vocab, scale, (const T*)pairs, buckets, mul_prev, mul_cur, last_token, write_state,              \
+                       (const T*)places, n_places, positions, q_start, seq_of_token, slot_ids, n_seqs, n_slots, status)
+  if (dtype == 0) SUM(float);
+  if (dtype == 1) SUM(__nv_bfloat16);
+#undef SUM
+  return kRefusedDtype;
 }
 
 extern "C" int leone_embedding(int dtype, const void* table, const int* ids, float* out, int n,

@@ -6,6 +6,9 @@
 //     S <- S + k_t u^T
 //     o_t = S^T q_t                               (the read-out sees the token's own write)
 //
+// or with a decay per key channel (CHANNEL): g_t = exp(-exp(A_log_h) softplus(z_t)), one z per head and row of S, and
+// S <- diag(g_t) S.
+//
 // q and k arrive as activations (after their convolution and silu) of `kv_heads` heads; the kernel makes
 // them unit vectors per head, x / sqrt(sum x^2 + 1e-6), and multiplies q by `q_scale`; head h reads
 // q/k head h / (heads / kv_heads).  a_t and b_t are raw projections, one per head.  Everything here is
@@ -33,10 +36,10 @@ template <int P> __device__ __forceinline__ float part_sum(float v) {
   return v;
 }
 
-template <int DPT, int P>
+template <int DPT, int P, bool CHANNEL, typename TR>
 __global__ void __launch_bounds__(kDeltaThreads)
 gated_delta_kernel(const float* __restrict__ act, int lda, int q_off, int k_off, int v_off,
-                   const float* __restrict__ raw, int ldr, int a_off, int b_off,
+                   const TR* __restrict__ raw, int ldr, int a_off, int b_off, const float* __restrict__ zs, int ldz,
                    const float* __restrict__ a_log, const float* __restrict__ dt_bias, float q_scale,
                    float* __restrict__ out, int ldo, float* state, const int* __restrict__ q_start,
                    const int* __restrict__ slot_ids, int heads, int kv_heads, int dim, int vdim, int n_slots,
@@ -47,7 +50,8 @@ gated_delta_kernel(const float* __restrict__ act, int lda, int q_off, int k_off,
   constexpr int CW = 32 / P;                    // value columns per warp
   constexpr int COLS = CW * (kDeltaThreads / 32);
   extern __shared__ __align__(16) float smem[];
-  // two stages of: q [tokens][DIMP], k [tokens][DIMP], v [tokens][COLS], decay [tokens], beta [tokens]
+  // two stages of: q [tokens][DIMP], k [tokens][DIMP], v [tokens][COLS], decay [tokens], beta [tokens], and with
+  // CHANNEL decays [tokens][DIMP]
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int part = lane % P;
   const int col_local = warp * CW + lane / P;
@@ -69,11 +73,11 @@ gated_delta_kernel(const float* __restrict__ act, int lda, int q_off, int k_off,
     const int i = part + P * r;
     S[r] = (i < dim && col < vdim) ? st[(size_t)i * vdim + col] : 0.f;
   }
-  const float rate = expf(a_log[h]), bias = dt_bias[h];
+  const float rate = expf(a_log[h]), bias = CHANNEL ? 0.f : dt_bias[h];
   // The raw rows of the next 16 tokens are requested (cp.async, 4 bytes each: no alignment is asked of the
   // rows) before the current 16 are walked, so the walk hides their latency; stage = which half of the
   // doubled buffers holds the current tokens.
-  constexpr int kStage = kDeltaTokens * (2 * DIMP + COLS) + 2 * kDeltaTokens;
+  constexpr int kStage = kDeltaTokens * ((CHANNEL ? 3 : 2) * DIMP + COLS) + 2 * kDeltaTokens;
   auto request = [&](int tb, int stage) {
     const int nt = min(kDeltaTokens, t1 - tb);
     float* qd = smem + stage * kStage;
@@ -85,9 +89,14 @@ gated_delta_kernel(const float* __restrict__ act, int lda, int q_off, int k_off,
         const float* row = act + (size_t)(tb + tt) * lda + (size_t)kvh * dim + d;
         asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(qd + i)), "l"(row + q_off));
         asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(kd + i)), "l"(row + k_off));
+        if (CHANNEL)
+          asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(
+                           vd + kDeltaTokens * COLS + 2 * kDeltaTokens + i)),
+                       "l"(zs + (size_t)(tb + tt) * ldz + (size_t)h * dim + d));
       } else {
         qd[i] = 0.f;
         kd[i] = 0.f;
+        if (CHANNEL) vd[kDeltaTokens * COLS + 2 * kDeltaTokens + i] = 0.f;
       }
     }
     for (int i = tid; i < nt * COLS; i += kDeltaThreads) {
@@ -106,11 +115,21 @@ gated_delta_kernel(const float* __restrict__ act, int lda, int q_off, int k_off,
     float* kd = qd + kDeltaTokens * DIMP;
     float* gd = kd + kDeltaTokens * DIMP + kDeltaTokens * COLS;
     if (tid < nt) {
-      const float* row = raw + (size_t)(tb + tid) * ldr;
-      const float z = row[a_off + h] + bias;
-      const float sp = z > 20.f ? z : log1pf(expf(z));           // softplus
-      gd[tid] = expf(-rate * sp);
-      gd[kDeltaTokens + tid] = 1.f / (1.f + expf(-row[b_off + h]));
+      const TR* row = raw + (size_t)(tb + tid) * ldr;
+      if (!CHANNEL) {
+        const float z = to_float<TR>(row[a_off + h]) + bias;
+        const float sp = z > 20.f ? z : log1pf(expf(z));           // softplus
+        gd[tid] = expf(-rate * sp);
+      }
+      gd[kDeltaTokens + tid] = 1.f / (1.f + expf(-to_float<TR>(row[b_off + h])));
+    }
+    if (CHANNEL) {
+      float* cd = gd + 2 * kDeltaTokens;
+      for (int i = tid; i < nt * DIMP; i += kDeltaThreads) {
+        const float z = cd[i];
+        const float sp = z > 20.f ? z : log1pf(expf(z));
+        cd[i] = expf(-rate * sp);
+      }
     }
     for (int tt = warp; tt < nt; tt += kDeltaThreads / 32) {
       float sq = 0.f, sk = 0.f;
@@ -142,7 +161,8 @@ gated_delta_kernel(const float* __restrict__ act, int lda, int q_off, int k_off,
     const float* v_c = k_c + kDeltaTokens * DIMP;
     const float* g_c = v_c + kDeltaTokens * COLS;
     for (int tt = 0; tt < nt; ++tt) {
-      const float g = g_c[tt], beta = g_c[kDeltaTokens + tt], vj = v_c[tt * COLS + col_local];
+      const float g = CHANNEL ? 1.f : g_c[tt], beta = g_c[kDeltaTokens + tt], vj = v_c[tt * COLS + col_local];
+      const float* gg = g_c + 2 * kDeltaTokens + tt * DIMP + part;
       const float* kk = k_c + tt * DIMP + part;
       const float* qq = q_c + tt * DIMP + part;
       float kv[DPT];
@@ -150,6 +170,7 @@ gated_delta_kernel(const float* __restrict__ act, int lda, int q_off, int k_off,
 #pragma unroll
       for (int r = 0; r < DPT; ++r) {
         kv[r] = kk[P * r];
+        if (CHANNEL) S[r] *= gg[P * r];
         r4[r & 3] = fmaf(S[r], kv[r], r4[r & 3]);
       }
       const float dot = part_sum<P>((r4[0] + r4[1]) + (r4[2] + r4[3]));
@@ -157,7 +178,7 @@ gated_delta_kernel(const float* __restrict__ act, int lda, int q_off, int k_off,
       float o4[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
       for (int r = 0; r < DPT; ++r) {
-        S[r] = fmaf(g, S[r], kv[r] * u);
+        S[r] = CHANNEL ? fmaf(kv[r], u, S[r]) : fmaf(g, S[r], kv[r] * u);
         o4[r & 3] = fmaf(S[r], qq[P * r], o4[r & 3]);
       }
       const float o = part_sum<P>((o4[0] + o4[1]) + (o4[2] + o4[3]));
@@ -210,10 +231,11 @@ group_gate_norm_kernel(const float* __restrict__ o, int ldo, int heads, int vdim
 using namespace leone;
 
 // act: fp32 [n_tokens, lda] with the activations of q and k (kv_heads x dim each) and v (heads x vdim) at
-// the given column offsets; raw: fp32 [n_tokens, ldr] with one a and one b per head at theirs.
+// the given column offsets; raw: [n_tokens, ldr] in `raw_dtype` with one a and one b per head at theirs.
+// zs: fp32 [n_tokens, ldz], head h's decay logits (bias added) at columns h * dim, or null (a decay per head from a).
 // out: fp32 [n_tokens, ldo], head h at columns h * vdim.  state: fp32 [n_slots, heads, dim, vdim].
-extern "C" int leone_gated_delta(const float* act, int lda, int q_off, int k_off, int v_off, const float* raw, int ldr,
-                                 int a_off, int b_off, const float* a_log, const float* dt_bias, float q_scale,
+extern "C" int leone_gated_delta(const float* act, int lda, int q_off, int k_off, int v_off, int raw_dtype,
+                                 const void* raw, int ldr, int a_off, int b_off, const float* zs, int ldz, const float* a_log, const float* dt_bias, float q_scale,
                                  float* out, int ldo, float* state, const int* q_start, const int* slot_ids,
                                  int n_seqs, int heads, int kv_heads, int dim, int vdim, int n_slots, int* status,
                                  cudaStream_t stream) {
@@ -221,20 +243,28 @@ extern "C" int leone_gated_delta(const float* act, int lda, int q_off, int k_off
   if (heads <= 0 || kv_heads <= 0 || heads % kv_heads != 0 || dim <= 0 || vdim <= 0 || dim > 512 || heads > 65535 ||
       n_seqs > 65535)
     return kRefusedSize;
-#define DELTA(DPT, P)                                                                                                 \
+#define DELTA_AS(DPT, P, CHANNEL, TR)                                                                                 \
   {                                                                                                                   \
     constexpr int cols = (32 / P) * (kDeltaThreads / 32);                                                             \
-    const size_t smem = 2 * sizeof(float) * (size_t)(kDeltaTokens * (2 * DPT * P + cols) + 2 * kDeltaTokens);             \
+    const size_t smem = 2 * sizeof(float) * (size_t)(kDeltaTokens * ((CHANNEL ? 3 : 2) * DPT * P + cols) + 2 * kDeltaTokens); \
     static bool configured = false;                                                                                   \
     if (!configured && smem > 48 * 1024) {                                                                            \
-      cudaFuncSetAttribute(gated_delta_kernel<DPT, P>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);       \
+      cudaFuncSetAttribute(gated_delta_kernel<DPT, P, CHANNEL, TR>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
       configured = true;                                                                                              \
     }                                                                                                                 \
-    return launch_kernel(gated_delta_kernel<DPT, P>, dim3((vdim + cols - 1) / cols, heads, n_seqs),                   \
-                         dim3(kDeltaThreads), smem, stream, act, lda, q_off, k_off, v_off, raw, ldr, a_off, b_off,    \
-                         a_log, dt_bias, q_scale, out, ldo, state, q_start, slot_ids, heads, kv_heads, dim, vdim,     \
-                         n_slots, status);                                                                            \
+    return launch_kernel(gated_delta_kernel<DPT, P, CHANNEL, TR>, dim3((vdim + cols - 1) / cols, heads, n_seqs),      \
+                         dim3(kDeltaThreads), smem, stream, act, lda, q_off, k_off, v_off, (const TR*)raw, ldr, a_off, \
+                         b_off, zs, ldz, a_log, dt_bias, q_scale, out, ldo, state, q_start, slot_ids, heads, kv_heads, \
+                         dim, vdim, n_slots, status);                                                                 \
   }
+#define DELTA(DPT, P)                                                                                                 \
+  {                                                                                                                   \
+    if (zs == nullptr && raw_dtype == 0) DELTA_AS(DPT, P, false, float)                                               \
+    if (zs == nullptr) DELTA_AS(DPT, P, false, __nv_bfloat16)                                                         \
+    if (raw_dtype == 0) DELTA_AS(DPT, P, true, float)                                                                 \
+    DELTA_AS(DPT, P, true, __nv_bfloat16)                                                                             \
+  }
+  if (raw_dtype != 0 && raw_dtype != 1) return kRefusedDtype;
   // rows dealt to 16 lanes from 33 rows on: a token's cost is the latency of its chain of sums and shuffles,
   // not its multiply-adds (dim 128: 0.48 us a token with 16 lanes a column, 0.59 with 4), and two columns a warp
   // give a prompt of one sequence 8 blocks a head
@@ -244,6 +274,7 @@ extern "C" int leone_gated_delta(const float* act, int lda, int q_off, int k_off
   if (dim <= 128) DELTA(8, 16)
   if (dim <= 256) DELTA(16, 16)
   DELTA(16, 32)
+#undef DELTA_AS
 #undef DELTA
 }
 

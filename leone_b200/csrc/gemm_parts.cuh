@@ -63,6 +63,9 @@ struct GemmParams {
   // and u' = clamp(u, -limit, limit).  gate_plain: slope 1, no limit, shift and cubic 0 (SwiGLU).
   int gate_plain;
   float gate_slope, gate_limit, gate_shift, gate_cubic;
+  // One fp32 number per weight row added to its sums (before a gate, a residual or a norm after the product), or
+  // null.
+  const float* bias;
 };
 
 // Host side: the gate fields from an optional {slope, limit, shift, cubic} (null: SwiGLU).
@@ -108,6 +111,22 @@ __device__ __forceinline__ float gate_mul(const GemmParams& p, float g, float u)
   return __fdividef(g, 1.f + __expf(-z)) * (u + p.gate_shift);
 }
 
+// v[j] += bias[n + j] for 16 weight rows from n on, a multiple of 16 (every thread of a warp reads the same addresses).
+__device__ __forceinline__ void add_bias16(const GemmParams& p, float* v, int n) {
+  if (n + 16 <= p.N) {
+    const float4* b = reinterpret_cast<const float4*>(p.bias + n);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const float4 q = __ldg(b + j);
+      v[4 * j] += q.x; v[4 * j + 1] += q.y; v[4 * j + 2] += q.z; v[4 * j + 3] += q.w;
+    }
+  } else {
+#pragma unroll
+    for (int j = 0; j < 16; ++j)
+      if (n + j < p.N) v[j] += p.bias[n + j];
+  }
+}
+
 // Swapped orientation: the thread that owns weight row n finishes NC token columns
 // m0 + c .. m0 + c + NC - 1 whose sums are in v (r: the residual values, fetched by the caller
 // before anything is stored, because the residual may be the output itself).
@@ -119,6 +138,11 @@ __device__ __forceinline__ void finish_swapped(const GemmParams& p, float (&v)[N
   if (p.norm_in_ss != nullptr) {
 #pragma unroll
     for (int j = 0; j < NC; ++j) v[j] *= rs_s[c + j];
+  }
+  if (p.bias != nullptr) {
+    const float b = n < p.N ? p.bias[n] : 0.f;
+#pragma unroll
+    for (int j = 0; j < NC; ++j) v[j] += b;
   }
   if (p.epilogue == 3) {
     // rows come in groups of 32: 16 gate rows (lanes 0-15) then their 16 up rows (lanes 16-31).
@@ -207,6 +231,10 @@ __device__ __forceinline__ void finish_token_major32(const GemmParams& p, float 
                                                      bool residual_added = false) {
   if (m >= p.M || n >= p.N) return;
   const bool vec_ok = (p.ldc & 7) == 0;
+  if (p.bias != nullptr) {
+    add_bias16(p, v, n);
+    add_bias16(p, v + 16, n + 16);
+  }
   if (p.epilogue == 3) {                                 // 16 gate columns, then their 16 up columns
     __nv_bfloat16* orow = (__nv_bfloat16*)p.out + (size_t)m * p.ldc;
     const int col = n >> 1;
@@ -273,6 +301,7 @@ __device__ __forceinline__ void finish_token_major32(const GemmParams& p, float 
   }
 }
 
+
 // Token-major form: the thread that owns token row m finishes the tile's bn weight rows from n0
 // on (tile n_tile; bn a multiple of 16, of 32 with the SwiGLU epilogue), 16 at a time, from tensor
 // memory at taddr: the norm's factor before, the product's epilogue, and the operand and sum of
@@ -322,6 +351,10 @@ __device__ __forceinline__ void finish_token_major_row(const GemmParams& p, uint
       if (p.norm_in_ss != nullptr) {
 #pragma unroll
         for (int j = 0; j < 16; ++j) { g[j] *= rs; u[j] *= rs; }
+      }
+      if (p.bias != nullptr && n0 + c < p.N) {     // (rows come in whole groups of 32)
+        add_bias16(p, g, n0 + c);
+        add_bias16(p, u, n0 + c + 16);
       }
       const int col = (n0 + c) >> 1;
       if (m < p.M && n0 + c < p.N) {
@@ -381,6 +414,7 @@ __device__ __forceinline__ void finish_token_major_row(const GemmParams& p, uint
         for (int j = 0; j < 4; ++j) {
           v[4 * j] += r[j].x; v[4 * j + 1] += r[j].y; v[4 * j + 2] += r[j].z; v[4 * j + 3] += r[j].w;
         }
+        if (p.bias != nullptr) add_bias16(p, v, n0 + i * 16);
         if (row_ok) {
 #pragma unroll
           for (int j = 0; j < 4; ++j)
@@ -399,6 +433,7 @@ __device__ __forceinline__ void finish_token_major_row(const GemmParams& p, uint
 #pragma unroll
         for (int j = 0; j < 16; ++j) v[j] *= rs;
       }
+      if (p.bias != nullptr) add_bias16(p, v, n);
       const size_t o = (size_t)m * p.ldc + n;
       const bool full = n + 16 <= p.N && vec_ok;
       if (p.epilogue == 0) {

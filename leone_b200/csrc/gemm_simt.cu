@@ -8,7 +8,8 @@
 // does not depend on what else is in the batch.
 //
 // Epilogues: 0 store in the input type; 1 store fp32; 2 store fp32 = acc + residual
-// (residual may alias the output: each element is read then written by one thread).
+// (residual may alias the output: each element is read then written by one thread).  bias: fp32 [N] added to
+// the sums before them, or null.
 #include "common.cuh"
 
 namespace leone {
@@ -18,7 +19,7 @@ constexpr int BM = 64, BN = 64, BK = 16;
 template <typename T, int EPI>
 __global__ void __launch_bounds__(256)
 gemm_simt_kernel(const T* __restrict__ A, const T* __restrict__ W, void* Cv,
-                 const float* residual, int M, int N, int K, int lda, int ldw, int ldc) {
+                 const float* residual, const float* __restrict__ bias, int M, int N, int K, int lda, int ldw, int ldc) {
   __shared__ float As[BK][BM + 4];
   __shared__ float Ws[BK][BN + 4];
   const int tid = threadIdx.x;
@@ -65,6 +66,7 @@ gemm_simt_kernel(const T* __restrict__ A, const T* __restrict__ W, void* Cv,
       const int n = n0 + tx * 4 + j;
       if (n >= N) continue;
       const size_t o = (size_t)m * ldc + n;
+      if (bias != nullptr) acc[i][j] += bias[n];
       if (EPI == 0) ((T*)Cv)[o] = from_float<T>(acc[i][j]);
       else if (EPI == 1) ((float*)Cv)[o] = acc[i][j];
       else ((float*)Cv)[o] = acc[i][j] + residual[o];
@@ -77,15 +79,15 @@ gemm_simt_kernel(const T* __restrict__ A, const T* __restrict__ W, void* Cv,
 using namespace leone;
 
 extern "C" int leone_gemm_simt(int dtype, int epilogue, const void* a, const void* w, void* c,
-                               const float* residual, int m, int n, int k, int lda, int ldw,
-                               int ldc, cudaStream_t stream) {
+                               const float* residual, const float* bias, int m, int n, int k, int lda,
+                               int ldw, int ldc, cudaStream_t stream) {
   if (m <= 0 || n <= 0) return 0;
   if (k <= 0 || lda < k || ldw < k || ldc < n) return kRefusedSize;
   if (epilogue == 2 && residual == nullptr) return kRefusedSize;
   dim3 grid((n + BN - 1) / BN, (m + BM - 1) / BM);
   if (grid.y > 65535) return kRefusedSize;
 #define LAUNCH(T, E)                                                                       \
-  gemm_simt_kernel<T, E><<<grid, 256, 0, stream>>>((const T*)a, (const T*)w, c, residual, m, \
+  gemm_simt_kernel<T, E><<<grid, 256, 0, stream>>>((const T*)a, (const T*)w, c, residual, bias, m, \
                                                    n, k, lda, ldw, ldc)
   if (dtype == 0) {
     if (epilogue == 0) LAUNCH(float, 0);

@@ -196,6 +196,111 @@ rms_norm_add_kernel(float* __restrict__ dst, const float* __restrict__ a, const 
   }
 }
 
+// The same for rows that vector accesses fit, with a row in registers (four columns a thread at a time), and one thing
+// more: `next_out` = the new dst row RMS-normed with `next_w` (fp32), for the sublayer that reads the stream next, so that a
+// norm on a sublayer's output and the norm before the sublayer after it are one pass over the row.
+template <typename T> __device__ __forceinline__ float4 row_load4(const T* p);
+template <> __device__ __forceinline__ float4 row_load4<float>(const float* p) { return *reinterpret_cast<const float4*>(p); }
+template <> __device__ __forceinline__ float4 row_load4<__nv_bfloat16>(const __nv_bfloat16* p) {
+  const uint2 r = *reinterpret_cast<const uint2*>(p);
+  return make_float4(__uint_as_float(r.x << 16), __uint_as_float(r.x & 0xffff0000u), __uint_as_float(r.y << 16),
+                     __uint_as_float(r.y & 0xffff0000u));
+}
+template <typename T> __device__ __forceinline__ void row_store4(T* p, float4 v);
+template <> __device__ __forceinline__ void row_store4<float>(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+template <> __device__ __forceinline__ void row_store4<__nv_bfloat16>(__nv_bfloat16* p, float4 v) {
+  const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+  uint2 r;
+  r.x = *reinterpret_cast<const uint32_t*>(&a);
+  r.y = *reinterpret_cast<const uint32_t*>(&b);
+  *reinterpret_cast<uint2*>(p) = r;
+}
+__device__ __forceinline__ float sq4(float4 v, float s) { return fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, s)))); }
+
+template <typename TW, typename TR, int R>
+__global__ void __launch_bounds__(256)
+rms_norm_add_vec_kernel(float* __restrict__ dst, const float* __restrict__ a, const TW* __restrict__ w_a,
+                        const float* __restrict__ b, const TW* __restrict__ w_b, int width, float coef, float eps,
+                        int accumulate, TR* __restrict__ rounded, const TW* __restrict__ w_then,
+                        const float* __restrict__ next_w, float next_eps, TR* __restrict__ next_out) {
+  pdl_trigger();
+  pdl_wait();
+  __shared__ float scratch[33];
+  const size_t base = (size_t)blockIdx.x * width;
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  float4 va[R], vb[R], vd[R];
+  float sa = 0.f, sb = 0.f;
+#pragma unroll
+  for (int i = 0; i < R; ++i) {
+    const int c = (threadIdx.x + i * blockDim.x) * 4;
+    const bool in = c < width;
+    va[i] = in ? row_load4<float>(a + base + c) : zero;
+    vb[i] = in && b != nullptr ? row_load4<float>(b + base + c) : zero;
+    vd[i] = in && accumulate ? row_load4<float>(dst + base + c) : zero;
+    sa = sq4(va[i], sa);
+    sb = sq4(vb[i], sb);
+  }
+  sa = block_sum(sa, scratch);
+  const float ra = coef / sqrtf(sa / (float)width + eps);
+  float rb = 0.f;
+  if (b != nullptr) {
+    sb = block_sum(sb, scratch);
+    rb = coef / sqrtf(sb / (float)width + eps);
+  }
+  float st = 0.f;
+#pragma unroll
+  for (int i = 0; i < R; ++i) {
+    const int c = (threadIdx.x + i * blockDim.x) * 4;
+    if (c < width) {
+      const float4 wa = row_load4<TW>(w_a + c);
+      float4 v = make_float4(va[i].x * ra * wa.x, va[i].y * ra * wa.y, va[i].z * ra * wa.z, va[i].w * ra * wa.w);
+      if (b != nullptr) {
+        const float4 wb = row_load4<TW>(w_b + c);
+        v.x = fmaf(vb[i].x * rb, wb.x, v.x);
+        v.y = fmaf(vb[i].y * rb, wb.y, v.y);
+        v.z = fmaf(vb[i].z * rb, wb.z, v.z);
+        v.w = fmaf(vb[i].w * rb, wb.w, v.w);
+      }
+      va[i] = v;
+      st = sq4(v, st);
+    }
+  }
+  float rt = 1.f;
+  if (w_then != nullptr) {
+    st = block_sum(st, scratch);
+    rt = 1.f / sqrtf(st / (float)width + eps);
+  }
+  float sn = 0.f;
+#pragma unroll
+  for (int i = 0; i < R; ++i) {
+    const int c = (threadIdx.x + i * blockDim.x) * 4;
+    if (c < width) {
+      float4 v = va[i];
+      if (w_then != nullptr) {
+        const float4 wt = row_load4<TW>(w_then + c);
+        v = make_float4(v.x * rt * wt.x, v.y * rt * wt.y, v.z * rt * wt.z, v.w * rt * wt.w);
+      }
+      v = make_float4(v.x + vd[i].x, v.y + vd[i].y, v.z + vd[i].z, v.w + vd[i].w);
+      row_store4<float>(dst + base + c, v);
+      if (rounded != nullptr) row_store4<TR>(rounded + base + c, v);
+      va[i] = v;
+      sn = sq4(v, sn);
+    }
+  }
+  if (next_out != nullptr) {
+    sn = block_sum(sn, scratch);
+    const float rn = 1.f / sqrtf(sn / (float)width + next_eps);
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+      const int c = (threadIdx.x + i * blockDim.x) * 4;
+      if (c < width) {
+        const float4 wn = row_load4<float>(next_w + c);
+        row_store4<TR>(next_out + base + c, make_float4(va[i].x * rn * wn.x, va[i].y * rn * wn.y, va[i].z * rn * wn.z, va[i].w * rn * wn.w));
+      }
+    }
+  }
+}
+
 // a[t, c] *= act(gate[t, c]): act 0 sigmoid, 1 silu.
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -336,6 +441,40 @@ extern "C" int leone_rms_norm_add(float* dst, const float* a, const void* w_a, c
   if (w_dtype == 1 && rounded_dtype == 0) NA(__nv_bfloat16, float);
   if (w_dtype == 1 && rounded_dtype == 1) NA(__nv_bfloat16, __nv_bfloat16);
 #undef NA
+  return kRefusedDtype;
+}
+
+// The same and, with next_out (in `rounded_dtype`, as `rounded` is) and next_w (fp32), the new dst rows RMS-normed for
+// their next reader; width a multiple of 4 up to 8,192, all rows 16-byte aligned.
+extern "C" int leone_rms_norm_add_next(float* dst, const float* a, const void* w_a, const float* b, const void* w_b,
+                                       int w_dtype, int n, int width, float coef, float eps, int accumulate, void* rounded,
+                                       int rounded_dtype, const void* w_then, const float* next_w, float next_eps,
+                                       void* next_out, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (width <= 0 || width % 4 != 0 || width > 8192 || (b != nullptr) != (w_b != nullptr) || (next_out != nullptr) != (next_w != nullptr))
+    return kRefusedSize;
+  if (((uintptr_t)dst | (uintptr_t)a | (uintptr_t)b | (uintptr_t)w_a | (uintptr_t)w_b | (uintptr_t)rounded |
+       (uintptr_t)w_then | (uintptr_t)next_w | (uintptr_t)next_out) & 15)
+    return kRefusedAlignment;
+  const int quads = width / 4;
+  const int threads = quads >= 256 ? 256 : (quads + 31) / 32 * 32, rows = (quads + threads - 1) / threads;
+#define NV(TW, TR, R)                                                                                                  \
+  return launch_kernel(rms_norm_add_vec_kernel<TW, TR, R>, dim3(n), dim3(threads), 0, stream, dst, a, (const TW*)w_a, b, \
+                       (const TW*)w_b, width, coef, eps, accumulate, (TR*)rounded, (const TW*)w_then, next_w, next_eps,  \
+                       (TR*)next_out)
+#define NVR(TW, TR)                 \
+  {                                 \
+    if (rows == 1) NV(TW, TR, 1);   \
+    if (rows == 2) NV(TW, TR, 2);   \
+    if (rows <= 4) NV(TW, TR, 4);   \
+    NV(TW, TR, 8);                  \
+  }
+  if (w_dtype == 0 && rounded_dtype == 0) NVR(float, float)
+  if (w_dtype == 0 && rounded_dtype == 1) NVR(float, __nv_bfloat16)
+  if (w_dtype == 1 && rounded_dtype == 0) NVR(__nv_bfloat16, float)
+  if (w_dtype == 1 && rounded_dtype == 1) NVR(__nv_bfloat16, __nv_bfloat16)
+#undef NVR
+#undef NV
   return kRefusedDtype;
 }
 

@@ -1,7 +1,7 @@
 // A short causal convolution over time on every channel, with the last taps - 1 inputs of every
 // sequence kept as fixed-size state between steps; and the minGRU recurrence.
 //
-//   leone_short_conv:        y_t[c] = (add_input & 1 ? x_t[c] : 0) + sum_j w[c, j] x_(t - taps + 1 + j)[c],
+//   leone_short_conv:        y_t[c] = (add_input & 1 ? x_t[c] : 0) + (bias ? bias[c] : 0) + sum_j w[c, j] x_(t - taps + 1 + j)[c],
 //                            then y * sigmoid(y) if add_input & 2,
 //                            inputs before a sequence's start are zero; an input before the step's
 //                            first token comes from the state
@@ -28,7 +28,7 @@ constexpr int kMaxTaps = 16;
 
 template <typename TI, typename TO>
 __global__ void __launch_bounds__(kConvThreads)
-short_conv_kernel(const TI* __restrict__ x, int ldx, const float* __restrict__ w, float* state,
+short_conv_kernel(const TI* __restrict__ x, int ldx, const float* __restrict__ w, const float* __restrict__ bias, float* state,
                   TO* __restrict__ out, int ldo, const int* __restrict__ q_start, const int* __restrict__ seq_of_token,
                   const int* __restrict__ slot_ids, int channels, int taps, int add_input, int update_state, int n_seqs,
                   int n_slots, int* status) {
@@ -48,7 +48,7 @@ short_conv_kernel(const TI* __restrict__ x, int ldx, const float* __restrict__ w
   }
   const int local = t - q_start[s];                 // tokens of the sequence in this step before this one
   float* st = state + (size_t)slot * (taps - 1) * channels;
-  float acc = 0.f;
+  float acc = bias != nullptr ? bias[c] : 0.f;
   for (int j = 0; j < taps; ++j) {
     const int back = taps - 1 - j;
     float v;
@@ -107,7 +107,8 @@ template <> struct ConvVec<__nv_bfloat16, 4> {
 
 template <typename TI, typename TO, int V, int kT>
 __global__ void __launch_bounds__(kConvThreads)
-short_conv_tile_kernel(const TI* __restrict__ x, int ldx, const float* __restrict__ w, const float* __restrict__ state,
+short_conv_tile_kernel(const TI* __restrict__ x, int ldx, const float* __restrict__ w, const float* __restrict__ bias,
+                       const float* __restrict__ state,
                        TO* __restrict__ out, int ldo, const int* __restrict__ q_start,
                        const int* __restrict__ seq_of_token, const int* __restrict__ slot_ids, int n_tokens, int channels,
                        int taps, int add_input, int n_seqs, int n_slots, int* status) {
@@ -120,6 +121,9 @@ short_conv_tile_kernel(const TI* __restrict__ x, int ldx, const float* __restric
   for (int j = 0; j < kT; ++j)
 #pragma unroll
     for (int e = 0; e < V; ++e) wt[j][e] = j < taps ? w[(size_t)(c + e) * taps + j] : 0.f;
+  float b0[V];
+#pragma unroll
+  for (int e = 0; e < V; ++e) b0[e] = bias != nullptr ? bias[c + e] : 0.f;
   pdl_wait();
   const int t_end = min(t0 + kConvTile, n_tokens);
   // Input r of the tile is row t0 - (taps - 1) + r of the step.  The rows are asked for before anything is
@@ -155,7 +159,7 @@ short_conv_tile_kernel(const TI* __restrict__ x, int ldx, const float* __restric
       if (t0 + i < t_end) {
         float acc[V];
 #pragma unroll
-        for (int e = 0; e < V; ++e) acc[e] = 0.f;
+        for (int e = 0; e < V; ++e) acc[e] = b0[e];
 #pragma unroll
         for (int j = 0; j < kT; ++j)
           if (j < taps) {
@@ -195,7 +199,7 @@ short_conv_tile_kernel(const TI* __restrict__ x, int ldx, const float* __restric
     const float* st = state + (size_t)slot * (taps - 1) * channels;
 #pragma unroll
     for (int e = 0; e < V; ++e) {
-      float acc = 0.f;
+      float acc = b0[e];
       for (int j = 0; j < taps; ++j) {
         const int back = taps - 1 - j;
         const float u = back <= local ? to_float<TI>(x[(size_t)(t - back) * ldx + c + e])
@@ -499,7 +503,7 @@ extern "C" int leone_add_scaled(float* x, const float* y, long long n, float sca
 
 // in_dtype / out_dtype: 0 float32, 1 bfloat16.
 // update_state: every sequence of the step brings one token, and the kernel moves the state on too.
-extern "C" int leone_short_conv(int in_dtype, int out_dtype, const void* x, int ldx, const float* w, float* state,
+extern "C" int leone_short_conv(int in_dtype, int out_dtype, const void* x, int ldx, const float* w, const float* bias, float* state,
                                 void* out, int ldo, const int* q_start, const int* seq_of_token, const int* slot_ids,
                                 int n_tokens, int channels, int taps, int add_input, int update_state, int n_seqs,
                                 int n_slots, int* status, cudaStream_t stream) {
@@ -517,14 +521,14 @@ extern "C" int leone_short_conv(int in_dtype, int out_dtype, const void* x, int 
   {                                                                                                                 \
     if (vec)                                                                                                        \
       return launch_kernel(short_conv_tile_kernel<TI, TO, 4, 4>, vec_grid, dim3(kConvThreads), 0, stream,           \
-                           (const TI*)x, ldx, w, state, (TO*)out, ldo, q_start, seq_of_token, slot_ids, n_tokens,  \
+                           (const TI*)x, ldx, w, bias, state, (TO*)out, ldo, q_start, seq_of_token, slot_ids, n_tokens,  \
                            channels, taps, add_input, n_seqs, n_slots, status);                                     \
     if (tiled)                                                                                                      \
       return launch_kernel(short_conv_tile_kernel<TI, TO, 1, kMaxTaps>, tile_grid, dim3(kConvThreads), 0, stream,   \
-                           (const TI*)x, ldx, w, state, (TO*)out, ldo, q_start, seq_of_token, slot_ids, n_tokens,  \
+                           (const TI*)x, ldx, w, bias, state, (TO*)out, ldo, q_start, seq_of_token, slot_ids, n_tokens,  \
                            channels, taps, add_input, n_seqs, n_slots, status);                                     \
     return launch_kernel(short_conv_kernel<TI, TO>, grid, dim3(kConvThreads), 0, stream, (const TI*)x, ldx, w,      \
-                         state, (TO*)out, ldo, q_start, seq_of_token, slot_ids, channels, taps, add_input,          \
+                         bias, state, (TO*)out, ldo, q_start, seq_of_token, slot_ids, channels, taps, add_input,          \
                          update_state, n_seqs, n_slots, status);                                                    \
   }
   if (in_dtype == 0 && out_dtype == 0) LAUNCH(float, float);

@@ -53,6 +53,7 @@ class StepContext:
         self.fixed_shapes = False      # True while a CUDA graph is captured or replayed
         self.stream_copy = None        # see Model._forward
         self.token_rows = {}
+        self.embedding_cache = None    # the embedding part's per-request state, if it asked for any
 
     def cache_view(self, run_position: int):
         """The cache of the layer at this position of the run order (None if it has none)."""

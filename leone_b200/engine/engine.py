@@ -34,6 +34,9 @@ _DTYPES = {"bfloat16": torch.bfloat16, "bf16": torch.bfloat16,
            "float32": torch.float32, "fp32": torch.float32, "f32": torch.float32}
 
 
+EMBEDDING = "embedding"      # stands for a run position where the embedding part's own state is named
+
+
 class StepError(RuntimeError):
     """A kernel reported a fault through the status word (bad token id, bad page, ...)."""
 
@@ -94,6 +97,8 @@ class Engine:
                 return None
             if isinstance(req, CacheBundle):
                 return ("bundle", {name: bind((*key, name), member) for name, member in req.members.items()})
+            if isinstance(req, PagedKV) and key[0] == EMBEDDING:
+                raise TypeError("an embedding part keeps fixed-size state only")
             if isinstance(req, PagedKV):
                 # the part says what it caches (widths, dtype, when pages go back); equal requests share a group
                 r = req.resolved(self.dtype)
@@ -113,6 +118,7 @@ class Engine:
                 return ("state", skey)
             raise TypeError(f"run position {key[0]}: unknown cache request {req!r}")
 
+        self._embedding_binding = bind((EMBEDDING,), self.model.embedding.cache_request())
         for pos, (req, source) in enumerate(plan):
             if source is not None:
                 self._run_source[pos] = source
@@ -279,6 +285,7 @@ class Engine:
                                       self.page_tokens, writes, per_row)
             return StateView(self._run_state[binding[1]], writes)
 
+        ctx.embedding_cache = view(self._embedding_binding, True)
         for pos in range(len(self.spec.run_order)):
             src = self._run_source.get(pos, pos)
             cache = view(self._run_binding.get(src), pos not in self._run_source)

@@ -1,2 +1,2 @@
 """Built-in architectures.  Importing this package registers them."""
-from . import kakirax, malapel, qwen3, sakinex, sarizen, ziginex  # noqa: F401
+from . import gulipel, kakirax, malapel, qwen3, sakinex, sarizen, ziginex  # noqa: F401

@@ -64,10 +64,13 @@ def _need(cond: bool, msg: str) -> None:
 
 
 class PreparedMatrix:
-    """A weight matrix ``[out, in]`` with what the kernels precompute for it."""
+    """A weight matrix ``[out, in]`` with what the kernels precompute for it, and the bias ``[out]`` (fp32, or
+    None) that every product with it adds to its sums."""
 
-    def __init__(self, weight: torch.Tensor):
+    def __init__(self, weight: torch.Tensor, bias: Optional[torch.Tensor] = None):
         self.weight = weight
+        self.bias = None if bias is None else bias.float().contiguous()
+        _need(bias is None or self.bias.shape == (weight.shape[0],), "a bias has one number per row of its matrix")
         self.out_features, self.in_features = weight.shape
         self.tma = None           # tensor map for the tensor-core kernel, made on first use
 
@@ -145,15 +148,18 @@ class CudaOps:
         """Device memory the ops allocate for themselves beyond the runtime's named buffers."""
         return self.fast.scratch_bytes() if self.fast is not None else 0
 
-    def prepare_matrix(self, w: torch.Tensor) -> PreparedMatrix:
+    def prepare_matrix(self, w: torch.Tensor, bias: Optional[torch.Tensor] = None) -> PreparedMatrix:
         _need(w.dim() == 2 and w.is_contiguous(), "a weight matrix must be contiguous [out, in]")
-        return PreparedMatrix(w)
+        return PreparedMatrix(w, bias)
 
-    def prepare_gate_up(self, gate: torch.Tensor, up: torch.Tensor) -> PreparedMatrix:
-        _need(gate.shape == up.shape, "gate and up matrices differ in shape")
+    def prepare_gate_up(self, gate: torch.Tensor, up: torch.Tensor, gate_bias: Optional[torch.Tensor] = None,
+                        up_bias: Optional[torch.Tensor] = None) -> PreparedMatrix:
+        """``gate_bias`` and ``up_bias``: added to the two products before the gate (both or neither)."""
+        _need(gate.shape == up.shape and (gate_bias is None) == (up_bias is None), "gate and up matrices differ in shape")
         if self.fast is not None:
-            return self.fast.prepare_gate_up(gate, up)
-        m = PreparedMatrix(torch.cat([gate, up], dim=0).contiguous())
+            return self.fast.prepare_gate_up(gate, up, gate_bias, up_bias)
+        m = PreparedMatrix(torch.cat([gate, up], dim=0).contiguous(),
+                           None if gate_bias is None else torch.cat([gate_bias, up_bias]))
         m.gate_up_layout = "stacked"
         return m
 
@@ -167,6 +173,28 @@ class CudaOps:
         _check(self.core.leone_embedding(_dt(table.dtype), _ptr(table), _ptr(ids), _ptr(out), n,
                                          hidden, table.shape[0], c_float(scale), _ptr(status), self._stream()),
                "embedding")
+
+    def embedding_sum(self, ctx, table, out, scale=1.0, pairs=None, buckets=0, mul_prev=0, mul_cur=0, last_token=None,
+                      write_state=True, places=None):
+        """``out[t] = scale * table[id_t] + pairs[row_t] + places[position_t]`` for the step's tokens, with ``row_t =
+        (previous id * mul_prev + id_t * mul_cur) mod buckets``, or ``buckets`` at a sequence's first position; ``pairs``
+        ``[buckets + 1, hidden]`` and ``places`` ``[positions, hidden]`` may be None.  ``last_token``: the sequences'
+        state, ``[slots, 1]`` 32-bit words that hold a token id each (read for a sequence's first token of the
+        step, left as the step's last token)."""
+        n, hidden = out.shape
+        _need(out.dtype == torch.float32 and out.is_contiguous() and ctx.token_ids.numel() == n, "embedding_sum output")
+        for t in (table, pairs, places):
+            _need(t is None or (t.dtype == table.dtype and t.is_contiguous() and t.shape[1] == hidden), "embedding_sum tables")
+        if pairs is not None:
+            _need(pairs.shape[0] == buckets + 1 and last_token is not None and last_token.is_contiguous()
+                  and last_token.element_size() == 4 and last_token.numel() == last_token.shape[0], "embedding_sum pairs/state")
+        self.launches += 1
+        _check(self.core.leone_embedding_sum(
+            _dt(table.dtype), _ptr(table), _ptr(ctx.token_ids), _ptr(out), n, hidden, table.shape[0], c_float(scale),
+            _ptr(pairs), int(buckets), ctypes.c_longlong(mul_prev), ctypes.c_longlong(mul_cur), _ptr(last_token),
+            1 if write_state else 0, _ptr(places), 0 if places is None else places.shape[0], _ptr(ctx.positions),
+            _ptr(ctx.q_start), _ptr(ctx.seq_of_token), _ptr(ctx.slot_ids), ctx.n_seqs,
+            0 if last_token is None else last_token.shape[0], _ptr(ctx.status), self._stream()), "embedding_sum")
 
     def logit_post(self, logits, scale: float = 1.0, soft_cap: Optional[float] = None):
         """In place: ``logits * scale``, then ``cap * tanh(. / cap)`` if a soft cap is given."""
@@ -207,12 +235,12 @@ class CudaOps:
         _check(self.core.leone_layer_norm(_ptr(x), _ptr(rows), _ptr(weight), _ptr(bias), _dt(weight.dtype), _ptr(out),
                                           _dt(out.dtype), n_out, hidden, c_float(eps), self._stream()), "layer_norm")
 
-    def _gemm_simt(self, x, w, out, epilogue, residual):
+    def _gemm_simt(self, x, w, out, epilogue, residual, bias=None):
         m, k = x.shape
         n = w.shape[0]
         self.launches += 1
         _check(self.core.leone_gemm_simt(_dt(x.dtype), epilogue, _ptr(x), _ptr(w), _ptr(out),
-                                         _ptr(residual), m, n, k, x.stride(0), w.stride(0),
+                                         _ptr(residual), _ptr(bias), m, n, k, x.stride(0), w.stride(0),
                                          out.stride(0), self._stream()), "gemm_simt")
 
     def linear_fuses_norm(self, n_tokens: int, w: PreparedMatrix) -> bool:
@@ -278,7 +306,7 @@ class CudaOps:
         if self.fast is not None and self.fast.linear(x, w, out, epilogue, residual):
             self.launches += 1
             return
-        self._gemm_simt(x, w.weight, out, epilogue, residual)
+        self._gemm_simt(x, w.weight, out, epilogue, residual, w.bias)
 
     def linear_swiglu(self, x, w_gate_up: PreparedMatrix, out, norm_in=None, gate_shape=None):
         """``out = silu(x @ gate.T) * (x @ up.T)`` for a matrix from ``prepare_gate_up``.
@@ -302,7 +330,7 @@ class CudaOps:
             return
         _need(getattr(w_gate_up, "gate_up_layout", None) == "stacked", "gate/up layout")
         scratch = self._scratch("gate_up", m, 2 * inter, x.dtype)
-        self._gemm_simt(x, w_gate_up.weight, scratch, 0, None)
+        self._gemm_simt(x, w_gate_up.weight, scratch, 0, None, w_gate_up.bias)
         self.launches += 1
         if gate_shape is None:
             _check(self.core.leone_swiglu(_dt(x.dtype), _ptr(scratch), _ptr(out), m, inter,
@@ -406,12 +434,14 @@ class CudaOps:
     _MASKS = {"causal": 0, "window": 1, "chunk": 2}
     _WEIGHTS = {"softmax": 0, "softmax_plus_one": 1, "sigmoid": 2}
 
-    def attention_prepare(self, ctx, qkv, n_q, n_kv, dk, dv, norm, q_w, k_w, eps, freqs, pairing, cache):
+    def attention_prepare(self, ctx, qkv, n_q, n_kv, dk, dv, norm, q_w, k_w, eps, freqs, pairing, cache, query_temp=None):
         """Norm (``None``, ``"per_head"`` or ``"whole"``; fp32 weights) and rotation (fp32
         ``freqs`` per pair or None) of q and k in place, and the step's keys and values into
         their pages (``csrc/attention_masked.cu``).  Row layout ``[q heads x dk | k heads x dk |
-        v heads x dv]``."""
+        v heads x dv]``.  ``query_temp = (coef, every)``: q at position p is also multiplied by ``1 + coef *
+        ln(floor((p + 1) / every) + 1)``."""
         n = qkv.shape[0]
+        coef, every = query_temp or (0.0, 0)
         _need(qkv.stride(1) == 1 and qkv.shape[1] == (n_q + n_kv) * dk + n_kv * dv, "attention_prepare: qkv layout")
         mode = {None: 0, "per_head": 1, "whole": 2}[norm]
         if mode:
@@ -436,8 +466,8 @@ class CudaOps:
         self.launches += 1
         _check(self.mixers.leone_attention_prepare(
             _dt(qkv.dtype), _ptr(qkv), qkv.stride(0), n, n_q, n_kv, dk, dv, mode, _ptr(q_w), _ptr(k_w), c_float(eps),
-            _ptr(freqs), rot, 1 if pairing == "adjacent" else 0, _ptr(ctx.positions), _ptr(ctx.seq_of_token),
-            *pool_args, _ptr(ctx.status), self._stream()), "attention_prepare")
+            _ptr(freqs), rot, 1 if pairing == "adjacent" else 0, c_float(coef), int(every), _ptr(ctx.positions),
+            _ptr(ctx.seq_of_token), *pool_args, _ptr(ctx.status), self._stream()), "attention_prepare")
 
     def attention_masked(self, ctx, qkv, out, n_q, n_kv, dk, dv, scale, mask, mask_size, weights, bias, cache):
         """Attention with a mask (``"causal"``, ``"window"``, ``"chunk"`` of ``mask_size``) and a
@@ -719,12 +749,15 @@ class CudaOps:
         return logits
 
     # -- short convolutions with state, the minGRU recurrence, pooled-window attention --------------
-    def short_conv(self, ctx, x, weight, state, out, add_input=False, update_state=False, activation=None):
+    def short_conv(self, ctx, x, weight, state, out, add_input=False, update_state=False, activation=None, bias=None):
         """``out_t = (x_t if add_input) + sum_j weight[:, j] x_(t - taps + 1 + j)`` on every channel,
         inputs before the step from ``state`` (fp32 ``[slots, taps - 1, channels]``), which is not
         changed (``csrc/short_conv.cu``) unless ``update_state``, which is for steps in which every
         sequence brings one token: the kernel then leaves the state as :meth:`short_conv_state`
-        would.  ``weight``: fp32 ``[channels, taps]``.  ``activation``: ``None`` or ``"silu"`` on the result."""
+        would.  ``weight``: fp32 ``[channels, taps]``.  ``activation``: ``None`` or ``"silu"`` on the result.
+        ``bias``: fp32 ``[channels]`` added to the sum, or None."""
+        _need(bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == weight.shape[0]),
+              "short_conv bias")
         _need(activation in (None, "silu"), f"short_conv: activation '{activation}'")
         _need(not update_state or ctx.decode_only, "short_conv: update_state is for steps of one token a sequence")
         n, channels = out.shape
@@ -735,7 +768,7 @@ class CudaOps:
                             and tuple(state.shape[1:]) == (taps - 1, channels)), "short_conv state")
         self.launches += 1
         _check(self.mixers.leone_short_conv(
-            _dt(x.dtype), _dt(out.dtype), _ptr(x), x.stride(0), _ptr(weight), _ptr(state), _ptr(out), out.stride(0),
+            _dt(x.dtype), _dt(out.dtype), _ptr(x), x.stride(0), _ptr(weight), _ptr(bias), _ptr(state), _ptr(out), out.stride(0),
             _ptr(ctx.q_start), _ptr(ctx.seq_of_token), _ptr(ctx.slot_ids), n, channels, taps,
             (1 if add_input else 0) | (2 if activation == "silu" else 0), 1 if update_state else 0, ctx.n_seqs, state.shape[0] if state is not None else 0, _ptr(ctx.status),
             self._stream()), "short_conv")
@@ -918,10 +951,13 @@ class CudaOps:
         self.launches += 1
         _check(self.mixers.leone_zero(_ptr(t), ctypes.c_longlong(t.numel() * t.element_size()), self._stream()), "zero")
 
-    def rms_norm_add(self, dst, a, w_a, eps, b=None, w_b=None, coef=1.0, accumulate=True, rounded=None, then=None):
+    def rms_norm_add(self, dst, a, w_a, eps, b=None, w_b=None, coef=1.0, accumulate=True, rounded=None, then=None,
+                     following=None):
         """``dst (+)= coef * (rms_norm(a) * w_a [+ rms_norm(b) * w_b])``: fp32 rows, each source normed over
         its own row; ``rounded``: also the new ``dst`` in another dtype (the stream for its next reader).
-        ``then``: a weight; the combination is itself RMS-normed with it (same eps) before it is added."""
+        ``then``: a weight; the combination is itself RMS-normed with it (same eps) before it is added.
+        ``following = (weight, eps, out)``: also ``out = rms_norm(new dst) * weight`` (fp32 weight), the norm before
+        the next reader of the stream."""
         n, width = dst.shape
         _need(dst.dtype == torch.float32 and dst.is_contiguous() and a.dtype == torch.float32 and a.is_contiguous()
               and a.shape == dst.shape and w_a.numel() == width and w_a.is_contiguous(), "rms_norm_add layout")
@@ -933,11 +969,23 @@ class CudaOps:
         if then is not None:
             _need(then.numel() == width and then.dtype == w_a.dtype and then.is_contiguous() and width <= 12000,
                   "rms_norm_add: the norm after the combination")
+        next_w, next_eps, next_out = following or (None, 0.0, None)
+        if following is not None:
+            _need(next_w.dtype == torch.float32 and next_w.is_contiguous() and next_w.numel() == width
+                  and next_out.shape == dst.shape and next_out.is_contiguous(), "rms_norm_add: the norm that follows")
+        side = rounded if rounded is not None else next_out
+        w_b = w_b if b is not None else None
+        args = (_ptr(dst), _ptr(a), _ptr(w_a), _ptr(b), _ptr(w_b), _dt(w_a.dtype), n, width, c_float(coef), c_float(eps),
+                1 if accumulate else 0, _ptr(rounded), 0 if side is None else _dt(side.dtype), _ptr(then))
         self.launches += 1
-        _check(self.mixers.leone_rms_norm_add(
-            _ptr(dst), _ptr(a), _ptr(w_a), _ptr(b), _ptr(w_b if b is not None else None), _dt(w_a.dtype), n, width,
-            c_float(coef), c_float(eps), 1 if accumulate else 0, _ptr(rounded),
-            0 if rounded is None else _dt(rounded.dtype), _ptr(then), self._stream()), "rms_norm_add")
+        if (width % 4 == 0 and width <= 8192 and (rounded is None or next_out is None or rounded.dtype == next_out.dtype)
+                and not any(t is not None and t.data_ptr() % 16 for t in (dst, a, w_a, b, w_b, rounded, then, next_w, next_out))):
+            _check(self.mixers.leone_rms_norm_add_next(*args, _ptr(next_w), c_float(next_eps), _ptr(next_out), self._stream()),
+                   "rms_norm_add")
+            return
+        _check(self.mixers.leone_rms_norm_add(*args, self._stream()), "rms_norm_add")
+        if following is not None:
+            self.rms_norm(dst, next_w, next_out, next_eps)
 
     def gate_rows(self, a, gate, act="sigmoid"):
         """In place: ``a[t, c] *= act(gate[t, c])`` (``"sigmoid"`` or ``"silu"``); both in one dtype."""
@@ -1018,22 +1066,25 @@ class CudaOps:
         return True
 
     def gated_delta(self, ctx, act, raw, out, state, a_log, dt_bias, heads, kv_heads, dim, vdim, q_off, k_off, v_off,
-                    a_off, b_off, q_scale):
+                    a_off, b_off, q_scale, channel_logits=None):
         """The gated delta rule over the step's tokens (``csrc/gated_delta.cu``).  ``act``: fp32 rows with the
-        activations of q, k (``kv_heads x dim``) and v (``heads x vdim``) at their offsets; ``raw``: fp32 rows with
-        one decay logit and one beta logit per head at ``a_off`` / ``b_off``; ``state``: fp32 ``[slots, heads,
-        dim, vdim]``; ``out``: fp32 ``[n, heads * vdim]``."""
+        activations of q, k (``kv_heads x dim``) and v (``heads x vdim``) at their offsets; ``raw``: rows (fp32 or bfloat16)
+        with one decay logit and one beta logit per head at ``a_off`` / ``b_off``; ``state``: fp32 ``[slots, heads,
+        dim, vdim]``; ``out``: fp32 ``[n, heads * vdim]``.  ``channel_logits``: fp32 ``[n, heads * dim]``, a decay
+        logit (bias added) per head and key channel instead of the one per head (``a_off`` and ``dt_bias`` unused)."""
         n = act.shape[0]
-        _need(act.dtype == torch.float32 and raw.dtype == torch.float32 and act.stride(1) == 1 and raw.stride(1) == 1
+        z = channel_logits
+        _need(z is None or (z.dtype == torch.float32 and z.stride(1) == 1 and z.shape == (n, heads * dim)), "gated_delta decays")
+        _need(act.dtype == torch.float32 and act.stride(1) == 1 and raw.stride(1) == 1
               and raw.shape[0] == n and out.dtype == torch.float32 and out.is_contiguous()
               and out.shape == (n, heads * vdim), "gated_delta layout")
         _need(state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (heads, dim, vdim)
-              and a_log.dtype == torch.float32 and a_log.numel() == heads and dt_bias.dtype == torch.float32
-              and dt_bias.numel() == heads, "gated_delta state/constants")
+              and a_log.dtype == torch.float32 and a_log.numel() == heads
+              and (z is not None or (dt_bias.dtype == torch.float32 and dt_bias.numel() == heads)), "gated_delta state/constants")
         self.launches += 1
         _check(self.mixers.leone_gated_delta(
-            _ptr(act), act.stride(0), q_off, k_off, v_off, _ptr(raw), raw.stride(0), a_off, b_off, _ptr(a_log),
-            _ptr(dt_bias), c_float(q_scale), _ptr(out), out.stride(0), _ptr(state), _ptr(ctx.q_start), _ptr(ctx.slot_ids),
+            _ptr(act), act.stride(0), q_off, k_off, v_off, _dt(raw.dtype), _ptr(raw), raw.stride(0), a_off, b_off,
+            _ptr(z), 0 if z is None else z.stride(0), _ptr(a_log), _ptr(dt_bias), c_float(q_scale), _ptr(out), out.stride(0), _ptr(state), _ptr(ctx.q_start), _ptr(ctx.slot_ids),
             ctx.n_seqs, heads, kv_heads, dim, vdim, state.shape[0], _ptr(ctx.status), self._stream()), "gated_delta")
 
     def group_gate_norm(self, o, weight, gate, out, eps, heads, vdim, act="sigmoid"):
@@ -1050,6 +1101,38 @@ class CudaOps:
             _dt(out.dtype), _ptr(o), o.stride(0), n, heads, vdim, _ptr(weight), _dt(weight.dtype), _ptr(gate),
             0 if gate is None else gate.stride(0), 1 if act == "silu" else 0, _ptr(out), out.stride(0), c_float(eps),
             self._stream()), "group_gate_norm")
+
+    def ssd(self, ctx, act, raw, out, state, a_log, dt_bias, d_skip, heads, groups, n_state, vdim, x_off, b_off, c_off, dt_off):
+        """The Mamba-2 recurrence over the step's tokens (``csrc/ssd.cu``).  ``act``: rows with the activations of x
+        (``heads x vdim``), B and C (``groups x n_state`` each) at their offsets; ``raw``: rows with one dt per head
+        at ``dt_off``; ``state``: fp32 ``[slots, heads, n_state, vdim]``; ``out``: fp32 ``[n, heads * vdim]``, the skip
+        ``D x`` included."""
+        n = act.shape[0]
+        _need(act.stride(1) == 1 and raw.stride(1) == 1 and raw.shape[0] == n and out.dtype == torch.float32
+              and out.stride(1) == 1 and out.shape == (n, heads * vdim), "ssd layout")
+        _need(state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (heads, n_state, vdim)
+              and all(t.dtype == torch.float32 and t.numel() == heads and t.is_contiguous() for t in (a_log, dt_bias, d_skip)),
+              "ssd state/constants")
+        _need(x_off + heads * vdim <= act.shape[1] and max(b_off, c_off) + groups * n_state <= act.shape[1]
+              and dt_off + heads <= raw.shape[1], "ssd columns")
+        self.launches += 1
+        _check(self.mixers.leone_ssd(
+            _dt(act.dtype), _ptr(act), act.stride(0), x_off, b_off, c_off, _dt(raw.dtype), _ptr(raw), raw.stride(0), dt_off,
+            _ptr(a_log), _ptr(dt_bias), _ptr(d_skip), _ptr(out), out.stride(0), _ptr(state), _ptr(ctx.q_start),
+            _ptr(ctx.slot_ids), ctx.n_seqs, heads, groups, n_state, vdim, state.shape[0], _ptr(ctx.status), self._stream()),
+            "ssd")
+
+    def grouped_gate_norm(self, y, z, weight, out, eps, groups):
+        """``out = rms_norm(y * silu(z)) * weight`` with a root mean square of its own for each of ``groups`` equal
+        parts of a row; ``y`` fp32, ``z`` and ``out`` fp32 or bfloat16, ``weight`` fp32."""
+        n, width = y.shape
+        _need(y.dtype == torch.float32 and y.stride(1) == 1 and z.shape == y.shape and z.stride(1) == 1
+              and out.shape == y.shape and out.stride(1) == 1 and width % groups == 0 and weight.dtype == torch.float32
+              and weight.numel() == width and weight.is_contiguous(), "grouped_gate_norm layout")
+        self.launches += 1
+        _check(self.mixers.leone_grouped_gate_norm(
+            _dt(out.dtype), _ptr(y), y.stride(0), _dt(z.dtype), _ptr(z), z.stride(0), _ptr(weight), _ptr(out), out.stride(0),
+            n, groups, width // groups, c_float(eps), self._stream()), "grouped_gate_norm")
 
     def experts_forward(self, x, w_gate, w_up, w_down, chosen, weight, top, scale_input, hidden, rt, identity=0,
                         fresh=False):

@@ -284,7 +284,7 @@ class FastKernels:
         return (False, *self.choose_splits(m, n, k))
 
     def _gemm(self, x, w, out, epilogue, residual, n_rows, splits=None, full_tiles=0, cluster=False,
-              norm_in=None, norm_out=None, token_major=None, gate_shape=None) -> bool:
+              norm_in=None, norm_out=None, token_major=None, gate_shape=None, bias=None) -> bool:
         """``splits=None`` lets :meth:`choose_splits` decide; otherwise tiles from
         ``full_tiles`` on are split ``splits`` ways, summed through a workspace or, with
         ``cluster``, inside a thread-block cluster.
@@ -316,14 +316,14 @@ class FastKernels:
             # pairs of SMs on tiles of 256 tokens (gemm_pair.cu)
             code = self.lib.leone_gemm_pair(_ptr(x), _ptr(w), _ptr(out), _ptr(residual), m, n_rows, k,
                                             x.stride(0), w.stride(0), out.stride(0), epilogue, width, splits, _ptr(ws),
-                                            _ptr(self.status), self.sm_count, *no, *ni, gs, self._stream())
+                                            _ptr(self.status), self.sm_count, *no, *ni, gs, _ptr(bias), self._stream())
             if code != 0:
                 raise RuntimeError(f"gemm_pair refused or failed with code {code} for m={m} n={n_rows} k={k}")
             return True
         code = self.lib.leone_gemm_tc(_ptr(x), _ptr(w), _ptr(out), _ptr(residual), m, n_rows, k,
                                       x.stride(0), w.stride(0), out.stride(0), epilogue, splits,
                                       full_tiles, _ptr(ws), _ptr(ct), _ptr(self.status), self.sm_count,
-                                      1 if cluster else 0, 1 if token_major else 0, *no, *ni, gs, self._stream())
+                                      1 if cluster else 0, 1 if token_major else 0, *no, *ni, gs, _ptr(bias), self._stream())
         if code != 0:
             raise RuntimeError(f"gemm_tc refused or failed with code {code} for m={m} n={n_rows} k={k} "
                                f"splits={splits} cluster={cluster} token_major={token_major}")
@@ -389,27 +389,33 @@ class FastKernels:
     def linear(self, x, w, out, epilogue, residual, norm_in=None, norm_out=None) -> bool:
         if not self._tc_ok(x, w.weight, out):
             return False
-        return self._gemm(x, w.weight, out, epilogue, residual, w.out_features, norm_in=norm_in, norm_out=norm_out)
+        return self._gemm(x, w.weight, out, epilogue, residual, w.out_features, norm_in=norm_in, norm_out=norm_out,
+                          bias=w.bias)
 
     # -- gate/up --------------------------------------------------------------------------
-    def prepare_gate_up(self, gate, up):
+    def prepare_gate_up(self, gate, up, gate_bias=None, up_bias=None):
         from .cuda import PreparedMatrix
         inter, hidden = gate.shape
         if gate.dtype == torch.bfloat16 and inter % 16 == 0 and hidden % 8 == 0 and self.use_tensor_cores:
             # groups of 32 rows: 16 gate rows, then the 16 up rows of the same columns
             stacked = torch.stack([gate.view(inter // 16, 16, hidden), up.view(inter // 16, 16, hidden)],
                                   dim=1).reshape(2 * inter, hidden).contiguous()
-            m = PreparedMatrix(stacked)
+            bias = None
+            if gate_bias is not None:
+                bias = torch.stack([gate_bias.view(inter // 16, 16), up_bias.view(inter // 16, 16)], dim=1).reshape(2 * inter)
+            m = PreparedMatrix(stacked, bias)
             m.gate_up_layout = "interleaved16"
             return m
-        m = PreparedMatrix(torch.cat([gate, up], dim=0).contiguous())
+        m = PreparedMatrix(torch.cat([gate, up], dim=0).contiguous(),
+                           None if gate_bias is None else torch.cat([gate_bias, up_bias]))
         m.gate_up_layout = "stacked"
         return m
 
     def linear_swiglu(self, x, w, out, norm_in=None, gate_shape=None) -> bool:
         if getattr(w, "gate_up_layout", None) != "interleaved16" or not self._tc_ok(x, w.weight, out):
             return False
-        return self._gemm(x, w.weight, out, 3, None, w.out_features, norm_in=norm_in, gate_shape=gate_shape)
+        return self._gemm(x, w.weight, out, 3, None, w.out_features, norm_in=norm_in, gate_shape=gate_shape,
+                          bias=w.bias)
 
     # -- attention ------------------------------------------------------------------------
     def decode_splits(self, n_seqs: int, n_kv: int, g: int, max_ctx: int) -> int:

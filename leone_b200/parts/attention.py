@@ -27,6 +27,9 @@ sum exp(s_j))``: one more member of score 0 without a value); ``"sigmoid"`` (``s
 b_head)`` for every seen key on its own, nothing normalised; ``b`` is the tensor ``bias_name``).
 ``gate_name``: an elementwise output gate: the heads' outputs, concatenated, times ``sigmoid(W_g x)`` (``W_g``:
 ``[heads * value_head_dim, hidden]``, rows of the fused input product) before ``W_o``.
+``bias = True``: q, k and v have biases (tensors ``<name>.b`` by default), added to their sums in the product.
+``query_temp``: ``{"coef", "every"}``: q at position ``p``, normed (and rotated), is multiplied by ``1 + coef *
+ln(floor((p + 1) / every) + 1)``.
 ``qk_norm = "whole"``: one RMS norm over all of a token's query heads together (weight
 ``[heads * head_dim]``, multiplied directly) and one over its key heads, before rotation.
 A position encoding that offers ``frequencies()`` instead of a table (``rotary_computed``): the
@@ -87,12 +90,17 @@ class Attention(Mixer):
         if self.mixed and self.weights != "softmax":
             raise ValueError("attention: temperature, cap, mixing and sink go with softmax weights")
         self.gate_name = params.get("gate_name")
+        temp = params.get("query_temp")
+        self.query_temp = (float(temp["coef"]), int(temp["every"])) if temp else None
+        if temp and self.query_temp[1] <= 0:
+            raise ValueError(f"attention: query_temp {temp}")
         self.scale = float(params.get("scale", 1.0 / math.sqrt(self.d)))
         pe_name = params.get("position_encoding")
         self.pos = (position_encodings or {}).get(pe_name) if pe_name else None
         if pe_name and self.pos is None:
             raise ValueError(f"attention names position encoding '{pe_name}' that the model lacks")
         self.names = {k: params.get(f"{k}_name", f"{k}_proj.weight") for k in ("q", "k", "v", "o")}
+        self.bias_names = [params.get(f"{k}_bias_name", f"{self.names[k]}.b") for k in ("q", "k", "v")] if params.get("bias") else []
         self.q_norm_name = params.get("q_norm_name", "q_norm.weight")
         self.k_norm_name = params.get("k_norm_name", "k_norm.weight")
         self.w_qkv = self.w_o = self.q_norm_w = self.k_norm_w = None
@@ -103,7 +111,7 @@ class Attention(Mixer):
         self.in_cols = -(-(self.gate_off + self.gate_rows) // 16) * 16 if self.gate_name else self.qkv_cols
         # the layer as the reference has it runs on the kernels tuned for it; anything else on the general ones
         self.general = (self.dv != self.d or self.mask == "chunk" or self.weights != "softmax" or self.norm_whole
-                        or self.mixed or bool(self.gate_name) or (self.pos is not None and hasattr(self.pos, "frequencies")))
+                        or self.mixed or bool(self.gate_name) or self.query_temp is not None or (self.pos is not None and hasattr(self.pos, "frequencies")))
         if self.general and self.pos is not None and not hasattr(self.pos, "frequencies"):
             raise ValueError("attention: the general kernels take a position encoding that offers its frequencies")
 
@@ -114,6 +122,9 @@ class Attention(Mixer):
                  WeightSpec(self.names["o"], (self.hidden, self.n_q * self.dv))]
         if self.gate_name:
             specs.append(WeightSpec(self.gate_name, (self.gate_rows, self.hidden)))
+        if self.bias_names:
+            specs += [WeightSpec(name, (rows,), role="vector", std=0.5) for name, rows in
+                      zip(self.bias_names, (self.n_q * self.d, self.n_kv * self.d, self.n_kv * self.dv))]
         if self.qk_norm:
             nq, nk = (self.n_q * self.d, self.n_kv * self.d) if self.norm_whole else (self.d, self.d)
             specs += [WeightSpec(self.q_norm_name, (nq,), role="norm", std=0.1),
@@ -135,7 +146,12 @@ class Attention(Mixer):
                 return torch.zeros((count, self.hidden), dtype=rows[0].dtype, device=rows[0].device)
             rows += [zeros(self.gate_off - self.qkv_cols), tensors[self.gate_name],
                      zeros(self.in_cols - self.gate_off - self.gate_rows)]
-        self.w_qkv = self.rt.ops.prepare_matrix(torch.cat(rows, dim=0).contiguous())
+        if self.bias_names:
+            bias = torch.zeros(self.in_cols, dtype=torch.float32, device=rows[0].device)
+            bias[:self.qkv_cols] = torch.cat([tensors[name].float() for name in self.bias_names])
+            self.w_qkv = self.rt.ops.prepare_matrix(torch.cat(rows, dim=0).contiguous(), bias)
+        else:
+            self.w_qkv = self.rt.ops.prepare_matrix(torch.cat(rows, dim=0).contiguous())
         self.w_o = self.rt.ops.prepare_matrix(tensors[self.names["o"]])
         self.q_norm_f32 = self.k_norm_f32 = None
         if self.qk_norm:
@@ -242,7 +258,8 @@ class Attention(Mixer):
         ops.attention_prepare(ctx, qkv, self.n_q, self.n_kv, self.d, self.dv,
                               "whole" if self.norm_whole else ("per_head" if self.qk_norm else None),
                               self.q_norm_f32 if self.qk_norm else None, self.k_norm_f32 if self.qk_norm else None,
-                              self.eps, freqs, pairing, cache if cache.writes else None)
+                              self.eps, freqs, pairing, cache if cache.writes else None,
+                              **({} if self.query_temp is None else {"query_temp": self.query_temp}))
         attn = rt.buffer("attn_out", n, self.n_q * self.dv, rt.dtype)
         size = self.window if self.mask == "window" else (self.chunk if self.mask == "chunk" else 0)
         if self.mixed:

@@ -166,6 +166,9 @@ class DeferredNorm:
     ss: Optional[torch.Tensor] = None
     parts: int = 0
     ready: bool = False
+    # the normed rows themselves, where the kernel that wrote the stream formed them on the way (then there is
+    # nothing left to fold: ``ready`` stays False and :meth:`materialize` gives these)
+    normed: Optional[torch.Tensor] = None
 
     def prepare(self, rt, parts: int) -> None:
         """Buffers for a step of ``n`` tokens: ``xn [n, size]`` and the partial sums ``ss
@@ -182,6 +185,8 @@ class DeferredNorm:
         self.ss = flat[:parts * n].view(parts, n)
 
     def materialize(self) -> torch.Tensor:
+        if self.normed is not None:
+            return self.normed
         return self.norm.forward(self.ctx, self.hidden)
 
 
@@ -309,6 +314,11 @@ class PositionEncoding(Part):
 class Embedding(Part):
     """Token ids → the fp32 residual stream.  Its tensors are named in full (no layer prefix).
     ``params`` always hold ``vocab_size`` and ``hidden_size``."""
+
+    def cache_request(self):
+        """Fixed-size state per request (a :class:`FixedState`, a bundle of them, or ``None``) for an embedding that
+        reads more than the step's own tokens; its view is ``ctx.embedding_cache``."""
+        return None
 
     def forward(self, ctx, hidden) -> None:
         """Fill ``hidden`` (fp32 ``[N, hidden_size]``) for the step's ``ctx.token_ids`` (at

@@ -31,7 +31,10 @@ class PreNormBlock(Block):
         """``pre``: this block's entry norm, already folded into the previous block's last
         product (or None); ``after``: the next block's entry norm for this block's last product
         to fold in.  Returns ``after`` if it was filled, else None."""
-        x = pre if pre is not None and pre.ready else self.mixer_norm.forward(ctx, hidden)
+        if pre is not None and pre.normed is not None:
+            x = pre.normed                # the kernel that wrote the stream formed the norm on the way
+        else:
+            x = pre if pre is not None and pre.ready else self.mixer_norm.forward(ctx, hidden)
         if self.feed_forward is None:
             if after is not None and getattr(self.mixer, "fuses_following_norm", False):
                 self.mixer.forward(ctx, cache, x, hidden, then=after)
@@ -120,6 +123,76 @@ class ParallelBlock(Block):
             xb = b.forward(ctx, hidden, out_name="normed_b")
         self.mixer.forward(ctx, cache, xa, hidden)
         self.feed_forward.forward(ctx, xb, hidden)
+
+
+@BLOCKS.register("sandwich_norm")
+class SandwichNormBlock(Block):
+    """``h += out_a(mixer(norm_a(h))); h += out_b(ffn(norm_b(h)))``: a norm before every sublayer and one on what it
+    gives back (extra parts ``mixer_out_norm`` and ``ffn_out_norm``), then, if the layer has one, a further part
+    ``after`` (registry ``feed_forward``) that reads the stream itself and adds to it on its own terms.  A layer
+    without a feed-forward (and without its norms) has the mixer's half only.
+
+    The kernel that adds a normed branch to the stream also leaves what the stream's next reader needs: the
+    norm before the next sublayer (of this block or, through ``after=``, the next one's first) or the
+    stream rounded to the run dtype for a part that reads it as it is."""
+
+    chains_norms = True
+    keeps_stream_copy = True
+
+    def __init__(self, mixer, feed_forward, mixer_norm, ffn_norm, mixer_out_norm=None, ffn_out_norm=None, after=None, **extra):
+        if mixer_norm is None or mixer_out_norm is None or extra or \
+                len({feed_forward is None, ffn_norm is None, ffn_out_norm is None}) != 1:
+            raise ValueError("the sandwich_norm arrangement is norm, mixer, norm and, optionally, norm, feed-forward, norm "
+                             "and a part after them: it takes exactly those parts")
+        for norm in (mixer_out_norm, ffn_out_norm):
+            if norm is not None and not hasattr(norm, "add_normed"):
+                raise ValueError("the sandwich_norm arrangement needs norms that can add a normed branch to the stream")
+        super().__init__(mixer, feed_forward, mixer_norm, ffn_norm)
+        self.mixer_out_norm, self.ffn_out_norm, self.after = mixer_out_norm, ffn_out_norm, after
+
+    def entry_norm(self, ctx, hidden):
+        return self.mixer_norm.defer(ctx, hidden, "mixer")
+
+    def _add(self, ctx, norm, part, args, hidden, rounded, following):
+        """Runs a sublayer and adds its normed result to the stream, in the sublayer's own last kernel where it can."""
+        rt = self.mixer.rt
+        folds = getattr(part, "adds_normed", None)
+        if folds is not None and folds(norm):
+            part.forward(*args, hidden, normed_by=norm, rounded=rounded, following=following)
+            return
+        branch = rt.buffer("sublayer_out", hidden.shape[0], hidden.shape[1], torch.float32)
+        PostNormBlock._run(part, rt, branch, *args)
+        norm.add_normed(ctx, branch, hidden, rounded=rounded, following=following)
+
+    def forward(self, ctx, cache, hidden, pre=None, after=None):
+        rt, n = self.mixer.rt, hidden.shape[0]
+        if pre is not None and (pre.normed is not None or (pre.ready and getattr(self.mixer, "accepts_deferred_norm", False))):
+            x = pre if pre.normed is None else pre.normed
+        else:
+            x = self.mixer_norm.forward(ctx, hidden)
+        # the norm of the block after this one, formed by the last kernel that writes the stream
+        last = None
+        if after is not None and hasattr(after.norm, "as_following"):
+            last = after.norm.as_following(n)
+        copy = None
+        if self.after is not None and rt.dtype != torch.float32:
+            copy = rt.buffer("stream_rounded", n, hidden.shape[1], rt.dtype)
+        if self.feed_forward is not None:
+            mid = self.ffn_norm.as_following(n) if hasattr(self.ffn_norm, "as_following") else None
+            self._add(ctx, self.mixer_out_norm, self.mixer, (ctx, cache, x), hidden, None, mid)
+            x = mid[2] if mid is not None else self.ffn_norm.forward(ctx, hidden)
+            part, norm, args = self.feed_forward, self.ffn_out_norm, (ctx, x)
+        else:
+            part, norm, args = self.mixer, self.mixer_out_norm, (ctx, cache, x)
+        ctx.stream_copy = None
+        if self.after is None:
+            self._add(ctx, norm, part, args, hidden, None, last)
+        else:
+            self._add(ctx, norm, part, args, hidden, copy, None)
+            self.after.forward(ctx, hidden if copy is None else copy, hidden, **({} if last is None else {"following": last}))
+        if last is not None:
+            after.normed = last[2]
+        return after if last is not None else None
 
 
 @BLOCKS.register("post_norm")

@@ -27,7 +27,7 @@ class SideBySide(Mixer):
         """True if ``forward(..., normed_by=norm)`` can fold the arrangement's norm on this mixer's output into
         its own combining kernel."""
         return (self.combine == "normed_mean" and len(self.branches) == 2 and getattr(norm, "eps", None) == self.eps
-                and getattr(norm, "weight", None) is not None and norm.weight.dtype == self.norm_weights[0].dtype
+                and getattr(norm, "weight_f32", None) is not None
                 and self.hidden <= 12000)
 
     def __init__(self, params, rt, position_encodings=None):
@@ -63,7 +63,7 @@ class SideBySide(Mixer):
         for _, part in self.branches:
             part.load({s.name: tensors[s.name] for s in part.weight_specs()})
         if self.combine == "normed_mean":
-            self.norm_weights = [tensors[name] for name in self.norm_names]
+            self.norm_weights = [tensors[name].float().contiguous() for name in self.norm_names]
 
     def weight_bytes(self):
         return sum(part.weight_bytes() for _, part in self.branches if hasattr(part, "weight_bytes"))
@@ -77,11 +77,12 @@ class SideBySide(Mixer):
     def cache_request(self):
         return CacheBundle({name: part.cache_request() for name, part in self.branches})
 
-    def forward(self, ctx, cache, x, hidden, fresh=False, normed_by=None, rounded=None):
+    def forward(self, ctx, cache, x, hidden, fresh=False, normed_by=None, rounded=None, following=None):
         """``normed_by``: a norm part whose ``weight`` and ``eps`` norm this mixer's whole result before it is
         added to ``hidden`` (the arrangement's norm on the mixer's output, folded into the combining kernel:
         only offered to a mixer that declares ``adds_normed``, and only taken with two branches of the normed
-        mean and the same eps); ``rounded``: also the new ``hidden`` in the run dtype."""
+        mean and the same eps); ``rounded``: also the new ``hidden`` in the run dtype; ``following``: the norm of the
+        new ``hidden``'s next reader (``as_following``), formed by the same kernel."""
         if self.combine == "sum":
             if fresh:
                 self.rt.ops.zero(hidden)
@@ -102,7 +103,7 @@ class SideBySide(Mixer):
         if normed_by is not None:
             # hidden += norm(mean of the normed branches): the two norms after one another in one kernel
             ops.rms_norm_add(hidden, outs[0], w[0], self.eps, b=outs[1], w_b=w[1], coef=coef, accumulate=True,
-                             rounded=rounded, then=normed_by.weight)
+                             rounded=rounded, then=normed_by.weight_f32, **({} if following is None else {"following": following}))
             return
         # the normed outputs two at a time: one pass over the rows for a pair of branches
         for i in range(0, len(outs), 2):

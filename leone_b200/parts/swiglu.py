@@ -10,6 +10,7 @@ The gate's shape is this part's own parameters, for gated layers of the same fam
 and ``u' = clamp(u, -limit, limit)``.  The defaults (``gate_slope = 1``, no ``limit``, ``up_shift`` and
 ``gate_cubic`` 0) are SwiGLU.  ``activation = "gelu_tanh"`` sets the slope and the cubic term to gelu's tanh form
 (GeGLU): ``z/2 (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))) = z sigmoid(2 sqrt(2/pi) z (1 + 0.044715 z^2))``.
+``bias = True``: all three projections have biases (tensors ``<name>.b`` by default), added to their sums in the products.
 """
 from __future__ import annotations
 
@@ -32,6 +33,9 @@ class SwiGLU(FeedForward):
         self.gate_name = params.get("gate_name", "gate_proj.weight")
         self.up_name = params.get("up_name", "up_proj.weight")
         self.down_name = params.get("down_name", "down_proj.weight")
+        self.bias = bool(params.get("bias", False))
+        self.bias_names = {k: params.get(f"{k}_bias_name", f"{n}.b") for k, n in
+                           (("gate", self.gate_name), ("up", self.up_name), ("down", self.down_name))}
         self.w_gate_up = None
         self.w_down = None
         activation = params.get("activation", "silu")
@@ -49,11 +53,22 @@ class SwiGLU(FeedForward):
             (slope, float("inf") if limit is None else float(limit), shift, cubic)
 
     def weight_specs(self):
-        return [WeightSpec(self.gate_name, (self.inter, self.hidden)),
-                WeightSpec(self.up_name, (self.inter, self.hidden)),
-                WeightSpec(self.down_name, (self.hidden, self.inter))]
+        specs = [WeightSpec(self.gate_name, (self.inter, self.hidden)),
+                 WeightSpec(self.up_name, (self.inter, self.hidden)),
+                 WeightSpec(self.down_name, (self.hidden, self.inter))]
+        if self.bias:
+            b = self.bias_names
+            specs += [WeightSpec(b["gate"], (self.inter,), role="vector", std=0.5),
+                      WeightSpec(b["up"], (self.inter,), role="vector", std=0.5),
+                      WeightSpec(b["down"], (self.hidden,), role="vector", std=0.5)]
+        return specs
 
     def load(self, tensors):
+        if self.bias:
+            gate_b, up_b, down_b = (tensors[self.bias_names[k]].float().contiguous() for k in ("gate", "up", "down"))
+            self.w_gate_up = self.rt.ops.prepare_gate_up(tensors[self.gate_name], tensors[self.up_name], gate_b, up_b)
+            self.w_down = self.rt.ops.prepare_matrix(tensors[self.down_name], down_b)
+            return
         self.w_gate_up = self.rt.ops.prepare_gate_up(tensors[self.gate_name], tensors[self.up_name])
         self.w_down = self.rt.ops.prepare_matrix(tensors[self.down_name])
 

@@ -45,7 +45,9 @@ class TokenGate(FeedForward):
     def scratch_bytes(self, max_tokens):
         return max_tokens * (self.dim * (4 + self.rt.dtype.itemsize) + self.hidden * 4)
 
-    def forward(self, ctx, x, hidden, rounded=None):
+    def forward(self, ctx, x, hidden, rounded=None, following=None):
+        """``rounded``: also the new stream in the run dtype; ``following``: the norm of its next reader
+        (``as_following``), formed by the kernel that adds this part's result."""
         rt, ops = self.rt, self.rt.ops
         n = hidden.shape[0]
         rows = ctx.token_rows.get(self.table)
@@ -57,4 +59,5 @@ class TokenGate(FeedForward):
         ops.gelu_gate(z, rows, self.offset, g)
         y = rt.buffer("token_gate_y", n, self.hidden, torch.float32)
         ops.linear(g, self.w_proj, y)
-        ops.rms_norm_add(hidden, y, self.norm_w, self.eps, rounded=rounded)
+        ops.rms_norm_add(hidden, y, self.norm_w, self.eps, rounded=rounded,
+                         **({} if following is None else {"following": following}))

@@ -20,11 +20,20 @@ class EmulatedOps:
         self.calls = []
 
     # -- weights ------------------------------------------------------------------------
-    def prepare_matrix(self, w):
+    def prepare_matrix(self, w, bias=None):
+        if bias is not None:
+            w = w.clone()
+            w.bias = bias.float()
         return w
 
-    def prepare_gate_up(self, gate, up):
-        return torch.cat([gate, up], dim=0).contiguous()
+    def prepare_gate_up(self, gate, up, gate_bias=None, up_bias=None):
+        return self.prepare_matrix(torch.cat([gate, up], dim=0).contiguous(),
+                                   None if gate_bias is None else torch.cat([gate_bias, up_bias]))
+
+    @staticmethod
+    def _product(x, w):
+        y = x.float() @ w.float().t()
+        return y if getattr(w, "bias", None) is None else y + w.bias
 
     def describe_status(self, word):
         return f"emulated status {word}"
@@ -32,6 +41,26 @@ class EmulatedOps:
     # -- kernels ------------------------------------------------------------------------
     def embedding(self, table, ids, out, status, scale=1.0):
         out.copy_(table[ids.long()].float() * scale)
+
+    def embedding_sum(self, ctx, table, out, scale=1.0, pairs=None, buckets=0, mul_prev=0, mul_cur=0, last_token=None,
+                      write_state=True, places=None):
+        ids = ctx.token_ids.long()
+        rows = table[ids].float() * scale
+        if places is not None:
+            rows = rows + places[ctx.positions.long()].float()
+        if pairs is not None:
+            words = last_token.view(torch.int32)
+            bounds, slots = ctx.q_start.tolist(), ctx.slot_ids.tolist()
+            for s, slot in enumerate(slots):
+                before = int(words[slot, 0])
+                for t in range(bounds[s], bounds[s + 1]):
+                    cur = int(ids[t])
+                    at = buckets if int(ctx.positions[t]) == 0 else (before * mul_prev + cur * mul_cur) % buckets
+                    rows[t] += pairs[at].float()
+                    before = cur
+                if write_state:
+                    words[slot, 0] = before
+        out.copy_(rows)
 
     def logit_post(self, logits, scale=1.0, soft_cap=None):
         logits.mul_(scale)
@@ -51,13 +80,13 @@ class EmulatedOps:
         out.copy_((y if bias is None else y + bias.float()).to(out.dtype))
 
     def linear(self, x, w, out, residual=None):
-        y = x.float() @ w.float().t()
+        y = self._product(x, w)
         if residual is not None:
             y = y + residual
         out.copy_(y.to(out.dtype))
 
     def linear_swiglu(self, x, w_gate_up, out, gate_shape=None):
-        y = x.float() @ w_gate_up.float().t()
+        y = self._product(x, w_gate_up)
         inter = y.shape[1] // 2
         if self.dtype != torch.float32:
             y = y.to(self.dtype).float()
@@ -69,7 +98,7 @@ class EmulatedOps:
     def convert(self, src, out):
         out.copy_(src.to(out.dtype))
 
-    def attention_prepare(self, ctx, qkv, n_q, n_kv, dk, dv, norm, q_w, k_w, eps, freqs, pairing, cache):
+    def attention_prepare(self, ctx, qkv, n_q, n_kv, dk, dv, norm, q_w, k_w, eps, freqs, pairing, cache, query_temp=None):
         n = qkv.shape[0]
         x = qkv.float()
         q, k = x[:, :n_q * dk], x[:, n_q * dk:(n_q + n_kv) * dk]
@@ -82,7 +111,11 @@ class EmulatedOps:
             q = q * torch.rsqrt((q * q).mean(dim=-1, keepdim=True) + eps) * q_w.float()
             k = k * torch.rsqrt((k * k).mean(dim=-1, keepdim=True) + eps) * k_w.float()
         pos = ctx.positions.long()
-        q = self._rotate(q, pos, freqs, 1.0, pairing).to(qkv.dtype)
+        q = self._rotate(q, pos, freqs, 1.0, pairing)
+        if query_temp is not None:
+            coef, every = query_temp
+            q = q * (1.0 + coef * torch.log(((pos + 1) // every + 1).float()))[:, None, None]
+        q = q.to(qkv.dtype)
         k = self._rotate(k, pos, freqs, 1.0, pairing).to(qkv.dtype)
         qkv[:, :n_q * dk] = q.reshape(n, -1)
         qkv[:, n_q * dk:(n_q + n_kv) * dk] = k.reshape(n, -1)
@@ -321,8 +354,10 @@ class EmulatedOps:
                 out[a + t] = (weight.t() * hist[t:t + taps]).sum(dim=0)
         return out + x if add_input else out
 
-    def short_conv(self, ctx, x, weight, state, out, add_input=False, update_state=False, activation=None):
+    def short_conv(self, ctx, x, weight, state, out, add_input=False, update_state=False, activation=None, bias=None):
         rows = self._conv_rows(ctx, x, weight, state, add_input)
+        if bias is not None:
+            rows = rows + bias
         if activation == "silu":
             rows = torch.nn.functional.silu(rows)
         out.copy_(rows.to(out.dtype))
@@ -422,7 +457,8 @@ class EmulatedOps:
     def zero(self, t):
         t.zero_()
 
-    def rms_norm_add(self, dst, a, w_a, eps, b=None, w_b=None, coef=1.0, accumulate=True, rounded=None, then=None):
+    def rms_norm_add(self, dst, a, w_a, eps, b=None, w_b=None, coef=1.0, accumulate=True, rounded=None, then=None,
+                     following=None):
         def normed(x, w):
             return x * torch.rsqrt((x * x).mean(dim=-1, keepdim=True) + eps) * w.float()
         v = normed(a, w_a)
@@ -434,6 +470,9 @@ class EmulatedOps:
         dst.copy_(dst + v if accumulate else v)
         if rounded is not None:
             rounded.copy_(dst.to(rounded.dtype))
+        if following is not None:
+            weight, next_eps, rows = following
+            self.rms_norm(dst, weight, rows, next_eps)
 
     def gate_rows(self, a, gate, act="sigmoid"):
         g = gate.float()
@@ -472,8 +511,9 @@ class EmulatedOps:
         out.copy_(res.reshape(n, n_q * dv).to(out.dtype))
 
     def gated_delta(self, ctx, act, raw, out, state, a_log, dt_bias, heads, kv_heads, dim, vdim, q_off, k_off, v_off,
-                    a_off, b_off, q_scale):
+                    a_off, b_off, q_scale, channel_logits=None):
         rep = heads // kv_heads
+        raw = raw.float()
         bounds, slots = ctx.q_start.tolist(), ctx.slot_ids.tolist()
 
         def unit(x):
@@ -485,12 +525,35 @@ class EmulatedOps:
                 k = unit(act[t, k_off:k_off + kv_heads * dim].view(kv_heads, dim)).repeat_interleave(rep, dim=0)
                 v = act[t, v_off:v_off + heads * vdim].view(heads, vdim)
                 beta = torch.sigmoid(raw[t, b_off:b_off + heads])
-                g = torch.exp(-torch.exp(a_log) * torch.nn.functional.softplus(raw[t, a_off:a_off + heads] + dt_bias))
-                st = g[:, None, None] * st
+                if channel_logits is None:
+                    z = (raw[t, a_off:a_off + heads] + dt_bias)[:, None]
+                else:
+                    z = channel_logits[t].view(heads, dim)
+                st = torch.exp(-torch.exp(a_log)[:, None] * torch.nn.functional.softplus(z))[:, :, None] * st
                 u = beta[:, None] * (v - torch.einsum("hdv,hd->hv", st, k))
                 st = st + k[:, :, None] * u[:, None, :]
                 out[t] = torch.einsum("hdv,hd->hv", st, q).reshape(-1)
             state[slot] = st
+
+    def ssd(self, ctx, act, raw, out, state, a_log, dt_bias, d_skip, heads, groups, n_state, vdim, x_off, b_off, c_off, dt_off):
+        rep, a = heads // groups, act.float()
+        bounds, slots = ctx.q_start.tolist(), ctx.slot_ids.tolist()
+        for s, slot in enumerate(slots):
+            st = state[slot]
+            for t in range(bounds[s], bounds[s + 1]):
+                x = a[t, x_off:x_off + heads * vdim].view(heads, vdim)
+                b = a[t, b_off:b_off + groups * n_state].view(groups, n_state).repeat_interleave(rep, dim=0)
+                c = a[t, c_off:c_off + groups * n_state].view(groups, n_state).repeat_interleave(rep, dim=0)
+                d = torch.nn.functional.softplus(raw[t, dt_off:dt_off + heads].float() + dt_bias)
+                st = torch.exp(-torch.exp(a_log) * d)[:, None, None] * st + (d[:, None] * b)[:, :, None] * x[:, None, :]
+                out[t] = (torch.einsum("hnv,hn->hv", st, c) + d_skip[:, None] * x).reshape(-1)
+            state[slot] = st
+
+    def grouped_gate_norm(self, y, z, weight, out, eps, groups):
+        v = y * torch.nn.functional.silu(z.float())
+        g = v.view(v.shape[0], groups, -1)
+        r = torch.rsqrt((g * g).mean(dim=-1, keepdim=True) + eps)
+        out.copy_(((g * r).reshape(v.shape) * weight).to(out.dtype))
 
     def gated_linear_attention(self, ctx, proj, gated, state, w2, w2_bias, norm_w, heads, dim, vdim, rank, tau, q_scale,
                                eps, q_off, k_off, v_off, u_off, gate_off, chunk=0, act="silu"):
