@@ -32,17 +32,6 @@ constexpr int kGmTokens = 16, kGmThreads = 256, kGmCols = 128;
 constexpr int kGmOPitch = kGmCols + 4;            // floats per token row of the read-out
 constexpr int kGmAPitch = kGmTokens + 8;          // bfloat16 per row of A
 
-// a, b as two packed bfloat16 terms each
-__device__ __forceinline__ void split_pair(float a, float b, uint32_t& hi, uint32_t& lo) {
-  hi = pack_bf16(a, b);
-  lo = pack_bf16(a - __uint_as_float(hi << 16), b - __uint_as_float(hi & 0xffff0000u));
-}
-
-__device__ __forceinline__ float exp2_fast(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
 __device__ __forceinline__ float log2_fast(float x) {
   float y;
   asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));

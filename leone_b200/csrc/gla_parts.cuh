@@ -28,10 +28,11 @@ struct GlaParams {
   int* status;
 };
 
-// The (sequence, chunk) pair a block works on, its token range, and whether it is the sequence's last.
+// The (sequence, chunk) pair a block works on, its token range, and whether it is the sequence's last (P: parameters with
+// chunk, n_seqs and q_start).
 struct GlaSpan { int seq, t0, t1, last; };
 
-__device__ __forceinline__ bool gla_span(const GlaParams& p, int z, GlaSpan& sp) {
+template <typename P> __device__ __forceinline__ bool gla_span(const P& p, int z, GlaSpan& sp) {
   if (p.chunk <= 0) {
     sp.seq = z;
     sp.t0 = p.q_start[z];

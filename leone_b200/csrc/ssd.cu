@@ -6,7 +6,8 @@
 //
 // x, B and C arrive as activations (after their convolution and silu), dt as a raw projection.  Everything here is
 // fp32.  The state is read from and written back to the request's state slot and the walk is token by token in the
-// same order whatever the cut; a step of one token per sequence (decode) is the same kernel.
+// same order whatever the cut; a step of one token per sequence (decode) is the same kernel.  Prompt portions of bfloat16
+// runs have a form of their own (ssd_mma.cu).
 //
 // A block owns (a slice of value columns, head, sequence).  A value column's rows are dealt to P lanes (row i belongs
 // to lane part i % P), DPT rows each in registers; the sum over rows is P-lane shuffles.  Tokens are staged 16 at a time,
@@ -201,7 +202,7 @@ extern "C" int leone_ssd(int act_dtype, const void* act, int lda, int x_off, int
     return kRefusedSize;
   if ((act_dtype | 1) != 1 || (raw_dtype | 1) != 1) return kRefusedDtype;
   SsdParams p = {act, lda, x_off, b_off, c_off, raw, ldr, dt_off, a_log, dt_bias, d_skip, out, ldo, state, q_start,
-                 slot_ids, n_seqs, heads, groups, n_state, vdim, n_slots, status};
+                 slot_ids, n_seqs, heads, groups, n_state, vdim, n_slots, status, 0, nullptr, nullptr};
 #define SSD_AS(TA, TR, DPT, P)                                                                                        \
   {                                                                                                                   \
     constexpr int cols = (32 / P) * (kSsdThreads / 32);                                                               \

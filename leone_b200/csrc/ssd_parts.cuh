@@ -19,6 +19,9 @@ struct SsdParams {
   const int* slot_ids;
   int n_seqs, heads, groups, n_state, vdim, n_slots;
   int* status;
+  int chunk;                   // 0: sequences are not cut
+  float* chunk_state;          // [chunks, heads, n_state, vdim]
+  float* chunk_decay;          // [chunks, heads, n_state], equal along n_state
 };
 
 // softplus(dt + bias), no clamp

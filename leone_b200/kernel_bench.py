@@ -441,6 +441,33 @@ def bench_gla(ops, tokens, batch, heads, dim, vdim, rank, chunk, reps, warmup):
     return row
 
 
+def bench_ssd(ops, tokens, batch, heads, groups, n_state, vdim, chunk, reps, warmup):
+    """The Mamba-2 recurrence (``CudaOps.ssd``): one prompt of ``tokens`` tokens, or with ``batch`` a decode step of that
+    many sequences."""
+    decode = batch > 0
+    seqs, q_len = (batch, 1) if decode else (1, tokens)
+    ctx = _step_of(seqs, q_len, q_len)
+    n, inner, bc = ctx.n_tokens, heads * vdim, groups * n_state
+    copies = 1 if not decode else max(1, int(300e6 // (seqs * heads * n_state * vdim * 4)) + 1)      # states larger together than L2
+    act = torch.randn((n, inner + 2 * bc), device=DEV).to(torch.bfloat16)
+    raw = torch.randn((n, 16 * -(-heads // 16)), device=DEV).to(torch.bfloat16)
+    out = torch.empty((n, inner), device=DEV)
+    states = [torch.zeros((seqs, heads, n_state, vdim), device=DEV) for _ in range(copies)]
+    a_log, dt_bias, skip = (torch.zeros(heads, device=DEV) for _ in range(3))
+    turn = {"i": 0}
+
+    def run():
+        turn["i"] = (turn["i"] + 1) % copies
+        ops.ssd(ctx, act, raw, out, states[turn["i"]], a_log, dt_bias, skip, heads, groups, n_state, vdim, 0, inner, inner + bc, 0,
+                chunk=chunk if q_len > chunk else 0)
+    ms = _time(run, reps, warmup, per_graph=copies if decode else 1)
+    moved = n * ((inner + 2 * bc + heads) * 2.0 + inner * 4.0) + 2.0 * seqs * heads * n_state * vdim * 4
+    row = dict(kernel="ssd", heads=heads, groups=groups, n_state=n_state, vdim=vdim, us=ms * 1e3, gbs=moved / ms / 1e6,
+               tflops=6.0 * n * inner * n_state / ms / 1e9)
+    row.update(dict(batch=batch) if decode else dict(tokens=tokens, chunk=chunk))
+    return row
+
+
 def bench_row_kernels(ops, tokens, width, reps, warmup):
     """Kernels that pass over rows once: the two norms of the fp32 stream, the output gate."""
     copies = max(1, min(64, int(300e6 // (tokens * width * 4)) + 1))
@@ -483,19 +510,20 @@ def bench_sampling(ops, rows, vocab, stages, reps, warmup):
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(prog="python -m leone_b200.kernel_bench")
     ap.add_argument("what", choices=["gemm", "decode-attention", "prefill-attention", "layer-shapes", "sampling",
-                                     "masked-attention", "pooled-attention", "conv-gru", "mixed-attention", "gated-delta", "gla",
+                                     "masked-attention", "pooled-attention", "conv-gru", "mixed-attention", "gated-delta", "gla", "ssd",
                                      "row-kernels"])
     ap.add_argument("--pool", type=int, default=64, help="pooled-attention: positions per pooled block")
     ap.add_argument("--taps", type=int, default=4, help="pooled-attention, conv-gru: taps of the short convolutions")
     ap.add_argument("--width", type=int, default=2048, help="conv-gru: channels; row-kernels: columns")
     ap.add_argument("--rank", type=int, default=16, help="gla: inner width of the decay's projection")
-    ap.add_argument("--chunk", type=int, default=None, help="conv-gru, gla: tokens per chunk of the recurrence (default: the part's)")
+    ap.add_argument("--groups", type=int, default=8, help="ssd: groups of heads that share B and C (--head-dim: state rows)")
+    ap.add_argument("--chunk", type=int, default=None, help="conv-gru, gla, ssd: tokens per chunk of the recurrence (default: the part's)")
     ap.add_argument("--mask", choices=["causal", "window", "chunk"], default="window")
     ap.add_argument("--mask-size", type=int, default=1024)
     ap.add_argument("--weights", choices=["softmax", "softmax_plus_one", "sigmoid"], default="sigmoid")
     ap.add_argument("--value-dim", type=int, default=0, help="masked-attention: value width (default: the head size)")
     ap.add_argument("--decode", action="store_true",
-                    help="masked-attention, pooled-attention, mixed-attention, gated-delta, gla, conv-gru: a decode step of --batch sequences")
+                    help="masked-attention, pooled-attention, mixed-attention, gated-delta, gla, ssd, conv-gru: a decode step of --batch sequences")
     ap.add_argument("--stages", default="top_k=40,top_p=0.95",
                     help="sampling: truncation stages in order, e.g. top_k=40,typical=0.9")
     ap.add_argument("--vocab", type=int, default=151936)
@@ -592,6 +620,9 @@ def main(argv=None) -> int:
     elif args.what == "gla":
         rows.append(bench_gla(ops, args.tokens, args.batch if args.decode else 0, args.heads, args.head_dim,
                               args.value_dim or args.head_dim, args.rank, args.chunk or 64, args.reps, args.warmup))
+    elif args.what == "ssd":
+        rows.append(bench_ssd(ops, args.tokens, args.batch if args.decode else 0, args.heads, args.groups, args.head_dim,
+                              args.value_dim or 64, args.chunk or 256, args.reps, args.warmup))
     elif args.what == "row-kernels":
         rows += bench_row_kernels(ops, args.tokens, args.width, args.reps, args.warmup)
     elif args.what == "conv-gru":

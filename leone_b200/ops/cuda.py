@@ -1102,11 +1102,13 @@ class CudaOps:
             0 if gate is None else gate.stride(0), 1 if act == "silu" else 0, _ptr(out), out.stride(0), c_float(eps),
             self._stream()), "group_gate_norm")
 
-    def ssd(self, ctx, act, raw, out, state, a_log, dt_bias, d_skip, heads, groups, n_state, vdim, x_off, b_off, c_off, dt_off):
+    def ssd(self, ctx, act, raw, out, state, a_log, dt_bias, d_skip, heads, groups, n_state, vdim, x_off, b_off, c_off, dt_off,
+            chunk=0):
         """The Mamba-2 recurrence over the step's tokens (``csrc/ssd.cu``).  ``act``: rows with the activations of x
         (``heads x vdim``), B and C (``groups x n_state`` each) at their offsets; ``raw``: rows with one dt per head
         at ``dt_off``; ``state``: fp32 ``[slots, heads, n_state, vdim]``; ``out``: fp32 ``[n, heads * vdim]``, the skip
-        ``D x`` included."""
+        ``D x`` included.  ``chunk`` > 0: prompt portions in bfloat16 are cut into chunks of that many tokens (a
+        multiple of 64) that run side by side (``csrc/ssd_mma.cu``)."""
         n = act.shape[0]
         _need(act.stride(1) == 1 and raw.stride(1) == 1 and raw.shape[0] == n and out.dtype == torch.float32
               and out.stride(1) == 1 and out.shape == (n, heads * vdim), "ssd layout")
@@ -1115,6 +1117,23 @@ class CudaOps:
               "ssd state/constants")
         _need(x_off + heads * vdim <= act.shape[1] and max(b_off, c_off) + groups * n_state <= act.shape[1]
               and dt_off + heads <= raw.shape[1], "ssd columns")
+        bf16 = act.dtype == torch.bfloat16 and raw.dtype == torch.bfloat16
+        if (bf16 and self.fast is not None and not ctx.decode_only and ctx.max_q_len >= 16
+                and os.environ.get("LEONE_NO_SSD_MMA", "0") != "1" and self.mixers.leone_ssd_mma_supported(n_state, vdim)
+                and act.stride(0) % 8 == 0 and act.data_ptr() % 16 == 0 and not any(o % 8 for o in (x_off, b_off, c_off))):
+            # prompt portions in bfloat16: 64 tokens at a time on tensor cores
+            n_chunks, chunk_state, chunk_decay = 0, None, None
+            if chunk > 0:
+                n_chunks = int(sum(-(-int(q) // chunk) for q in ctx.q_lens))
+                chunk_state = self._scratch("ssd_chunk_state", n_chunks, heads * n_state * vdim, torch.float32)
+                chunk_decay = self._scratch("ssd_chunk_decay", n_chunks, heads * n_state, torch.float32)
+            self.launches += 1 if chunk == 0 else 3
+            _check(self.mixers.leone_ssd_mma(
+                _ptr(act), act.stride(0), x_off, b_off, c_off, _ptr(raw), raw.stride(0), dt_off, _ptr(a_log), _ptr(dt_bias),
+                _ptr(d_skip), _ptr(out), out.stride(0), _ptr(state), _ptr(ctx.q_start), _ptr(ctx.slot_ids), ctx.n_seqs, heads,
+                groups, n_state, vdim, state.shape[0], chunk, n_chunks, _ptr(chunk_state), _ptr(chunk_decay),
+                _ptr(ctx.status), self._stream()), "ssd (tensor cores)")
+            return
         self.launches += 1
         _check(self.mixers.leone_ssd(
             _dt(act.dtype), _ptr(act), act.stride(0), x_off, b_off, c_off, _dt(raw.dtype), _ptr(raw), raw.stride(0), dt_off,

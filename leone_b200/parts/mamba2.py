@@ -81,7 +81,9 @@ class Mamba2(Mixer):
         return (self.cols * self.hidden + self.hidden * self.inner) * self.rt.dtype.itemsize
 
     def scratch_bytes(self, max_tokens):
-        return max_tokens * ((self.cols + self.conv_cols + self.inner) * self.rt.dtype.itemsize + self.inner * 4)
+        chunks = max_tokens // self.chunk_for(max_tokens) + 1
+        return max_tokens * ((self.cols + self.conv_cols + self.inner) * self.rt.dtype.itemsize + self.inner * 4) \
+            + chunks * self.heads * self.n_state * (self.vdim + 1) * 4
 
     def load_transient_bytes(self):
         return self.cols * self.hidden * self.rt.dtype.itemsize
@@ -89,6 +91,14 @@ class Mamba2(Mixer):
     def cache_request(self):
         return CacheBundle({"state": FixedState((self.heads, self.n_state, self.vdim)),
                             "conv": FixedState((self.taps - 1, self.conv_cols)) if self.taps > 1 else None})
+
+    def chunk_for(self, tokens):
+        """The longest chunk (a power of two from 64 to 512) that leaves about a block and a half for each of 148 SMs:
+        longer chunks move fewer states between the kernels, but an SM without a block does nothing."""
+        chunk = 64
+        while chunk < 512 and tokens * self.heads * -(-self.vdim // 64) >= 2 * chunk * 200:
+            chunk *= 2
+        return chunk
 
     def forward(self, ctx, cache, x, hidden, fresh=False):
         rt, ops = self.rt, self.rt.ops
@@ -104,9 +114,13 @@ class Mamba2(Mixer):
         ops.short_conv(ctx, raw, self.conv_w, conv_state, act, activation="silu", update_state=fused, bias=self.conv_b)
         if conv_state is not None and conv.writes and not fused:
             ops.short_conv_state(ctx, raw, conv_state)
+        # long portions run chunk-parallel
+        chunk = 0 if ctx.decode_only else self.chunk_for(n)
+        if ctx.max_q_len <= chunk:
+            chunk = 0
         y = rt.buffer("mamba_y", n, self.inner, torch.float32)
         ops.ssd(ctx, act, proj, y, state.state, self.a_log, self.dt_bias, self.d_skip, self.heads, self.groups, self.n_state,
-                self.vdim, x_off=0, b_off=self.inner, c_off=self.inner + self.bc, dt_off=self.dt_off)
+                self.vdim, x_off=0, b_off=self.inner, c_off=self.inner + self.bc, dt_off=self.dt_off, chunk=chunk)
         gated = rt.buffer("mamba_gated", n, self.inner, rt.dtype)
         ops.grouped_gate_norm(y, proj[:, :self.inner], self.norm_w, gated, self.eps, self.norm_groups)
         ops.linear(gated, self.w_o, hidden, residual=None if fresh else hidden)

@@ -535,7 +535,8 @@ class EmulatedOps:
                 out[t] = torch.einsum("hdv,hd->hv", st, q).reshape(-1)
             state[slot] = st
 
-    def ssd(self, ctx, act, raw, out, state, a_log, dt_bias, d_skip, heads, groups, n_state, vdim, x_off, b_off, c_off, dt_off):
+    def ssd(self, ctx, act, raw, out, state, a_log, dt_bias, d_skip, heads, groups, n_state, vdim, x_off, b_off, c_off, dt_off,
+            chunk=0):
         rep, a = heads // groups, act.float()
         bounds, slots = ctx.q_start.tolist(), ctx.slot_ids.tolist()
         for s, slot in enumerate(slots):

@@ -504,7 +504,8 @@ def test_ssd_kernels_against_the_plain_recurrence(heads, groups, n_state, vdim, 
         y, S = plain.ssd_recurrence(x, B, C, plain.softplus(raws[s][:, 3:].double() + dt_bias.double()), torch.exp(a_log.double()))
         want.append((y + skip.double()[None, :, None] * x).reshape(n, inner))
         states.append(S)
-    for dtype, switch, tol in ((torch.float32, "1", 3e-5), (torch.bfloat16, "0", 1e-4), (torch.bfloat16, "1", 3e-5)):
+    for dtype, switch, chunk, tol in ((torch.float32, "0", 0, 3e-5), (torch.bfloat16, "1", 0, 3e-5), (torch.bfloat16, "0", 0, 1e-4),
+                                      (torch.bfloat16, "0", 64, 1e-4), (torch.bfloat16, "0", 128, 1e-4)):
         monkeypatch.setenv("LEONE_NO_SSD_MMA", switch)
         ops = CudaOps("cuda:0", dtype)
         state = torch.randn(4, heads, n_state, vdim, generator=g).cuda()       # what a slot held before must not matter
@@ -519,16 +520,16 @@ def test_ssd_kernels_against_the_plain_recurrence(heads, groups, n_state, vdim, 
             raw = torch.cat([raws[s][done[s]:done[s] + cuts[s][step]] for s in live]).to(dtype).cuda()
             out = torch.zeros(sum(q_lens), inner, device="cuda:0")
             ops.ssd(ctx, act, raw, out, state, a_log.cuda(), dt_bias.cuda(), skip.cuda(), heads, groups, n_state, vdim,
-                    x_off=0, b_off=inner, c_off=inner + bc, dt_off=3)
+                    x_off=0, b_off=inner, c_off=inner + bc, dt_off=3, chunk=chunk if max(q_lens) > chunk else 0)
             assert int(ctx.status[0]) == 0
             for j, s in enumerate(live):
                 got[s][done[s]:done[s] + cuts[s][step]] = out[starts[j]:starts[j + 1]].cpu().double()
                 done[s] += cuts[s][step]
         for s in range(3):
             err = float((got[s] - want[s]).abs().max()) / float(want[s].abs().max())
-            assert err <= tol, (dtype, switch, s, err)
+            assert err <= tol, (dtype, switch, chunk, s, err)
             serr = float((state[slots[s]].cpu().double() - states[s]).abs().max()) / float(states[s].abs().max())
-            assert serr <= tol, (dtype, switch, s, "state", serr)
+            assert serr <= tol, (dtype, switch, chunk, s, "state", serr)
 
 
 @pytest.mark.gpu
