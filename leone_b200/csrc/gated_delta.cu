@@ -14,7 +14,7 @@
 // q/k head h / (heads / kv_heads).  a_t and b_t are raw projections, one per head.  Everything here is
 // fp32.  The state is read from and written back to the request's state slot, and the walk is token
 // by token in the same order whatever the cut, so a step of one token per sequence (decode) is the
-// same kernel.
+// same kernel.  Prompt portions of bfloat16 runs have a form of their own (gated_delta_mma.cu).
 //
 // A block owns (sequence, head, a slice of value columns).  A value column's rows are dealt to P
 // lanes (row i belongs to lane part i % P), DPT rows each in registers; the two sums over rows of a

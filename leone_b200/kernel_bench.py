@@ -390,9 +390,9 @@ def bench_mixed_attention(ops, tokens, batch, context, n_q, n_kv, dk, dv, mask, 
     return row
 
 
-def bench_gated_delta(ops, tokens, batch, heads, kv_heads, dim, vdim, reps, warmup):
-    """The gated delta rule's recurrence (``CudaOps.gated_delta``): one prompt of ``tokens`` tokens, or with
-    ``batch`` a decode step of that many sequences."""
+def bench_gated_delta(ops, tokens, batch, heads, kv_heads, dim, vdim, per_channel, reps, warmup):
+    """The gated delta rule's recurrence (``CudaOps.gated_delta``), with a decay per head or per key channel: one prompt of
+    ``tokens`` tokens, or with ``batch`` a decode step of that many sequences."""
     decode = batch > 0
     seqs, q_len = (batch, 1) if decode else (1, tokens)
     ctx = _step_of(seqs, q_len, q_len)
@@ -402,9 +402,10 @@ def bench_gated_delta(ops, tokens, batch, heads, kv_heads, dim, vdim, reps, warm
     out = torch.empty((n, hv), device=DEV)
     state = torch.zeros((seqs, heads, dim, vdim), device=DEV)
     a_log, dt_bias = torch.zeros(heads, device=DEV), torch.zeros(heads, device=DEV)
+    kw = {"channel_logits": torch.randn((n, heads * dim), device=DEV)} if per_channel else {}
     ms = _time(lambda: ops.gated_delta(ctx, act, raw, out, state, a_log, dt_bias, heads, kv_heads, dim, vdim, 0, qk, 2 * qk,
-                                       0, heads, dim ** -0.5), reps, warmup, per_graph=16 if decode else 1)
-    row = dict(kernel="gated_delta", heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, us=ms * 1e3,
+                                       0, heads, dim ** -0.5, **kw), reps, warmup, per_graph=16 if decode else 1)
+    row = dict(kernel="gated_delta", heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, per_channel=per_channel, us=ms * 1e3,
                us_per_token=ms * 1e3 / q_len, fp32_tflops=6.0 * n * heads * dim * vdim / ms / 1e9)
     if decode:
         row.update(batch=batch, gbs=2.0 * seqs * heads * dim * vdim * 4 / ms / 1e6)
@@ -516,6 +517,7 @@ def main(argv=None) -> int:
     ap.add_argument("--taps", type=int, default=4, help="pooled-attention, conv-gru: taps of the short convolutions")
     ap.add_argument("--width", type=int, default=2048, help="conv-gru: channels; row-kernels: columns")
     ap.add_argument("--rank", type=int, default=16, help="gla: inner width of the decay's projection")
+    ap.add_argument("--per-channel", action="store_true", help="gated-delta: a decay per key channel instead of one per head")
     ap.add_argument("--groups", type=int, default=8, help="ssd: groups of heads that share B and C (--head-dim: state rows)")
     ap.add_argument("--chunk", type=int, default=None, help="conv-gru, gla, ssd: tokens per chunk of the recurrence (default: the part's)")
     ap.add_argument("--mask", choices=["causal", "window", "chunk"], default="window")
@@ -615,8 +617,8 @@ def main(argv=None) -> int:
                                           args.kv_heads, args.head_dim, args.value_dim or args.head_dim, args.mask,
                                           args.mask_size, args.page_tokens, args.reps, args.warmup))
     elif args.what == "gated-delta":
-        rows.append(bench_gated_delta(CudaOps(DEV, torch.float32), args.tokens, args.batch if args.decode else 0, args.heads,
-                                      args.kv_heads, args.head_dim, args.value_dim or args.head_dim, args.reps, args.warmup))
+        rows.append(bench_gated_delta(ops, args.tokens, args.batch if args.decode else 0, args.heads, args.kv_heads,
+                                      args.head_dim, args.value_dim or args.head_dim, args.per_channel, args.reps, args.warmup))
     elif args.what == "gla":
         rows.append(bench_gla(ops, args.tokens, args.batch if args.decode else 0, args.heads, args.head_dim,
                               args.value_dim or args.head_dim, args.rank, args.chunk or 64, args.reps, args.warmup))

@@ -1067,7 +1067,8 @@ class CudaOps:
 
     def gated_delta(self, ctx, act, raw, out, state, a_log, dt_bias, heads, kv_heads, dim, vdim, q_off, k_off, v_off,
                     a_off, b_off, q_scale, channel_logits=None):
-        """The gated delta rule over the step's tokens (``csrc/gated_delta.cu``).  ``act``: fp32 rows with the
+        """The gated delta rule over the step's tokens (``csrc/gated_delta.cu``; prompt portions of bfloat16 runs:
+        ``csrc/gated_delta_mma.cu``).  ``act``: fp32 rows with the
         activations of q, k (``kv_heads x dim``) and v (``heads x vdim``) at their offsets; ``raw``: rows (fp32 or bfloat16)
         with one decay logit and one beta logit per head at ``a_off`` / ``b_off``; ``state``: fp32 ``[slots, heads,
         dim, vdim]``; ``out``: fp32 ``[n, heads * vdim]``.  ``channel_logits``: fp32 ``[n, heads * dim]``, a decay
@@ -1081,6 +1082,20 @@ class CudaOps:
         _need(state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (heads, dim, vdim)
               and a_log.dtype == torch.float32 and a_log.numel() == heads
               and (z is not None or (dt_bias.dtype == torch.float32 and dt_bias.numel() == heads)), "gated_delta state/constants")
+        if (self.fast is not None and not ctx.decode_only and ctx.max_q_len >= 16
+                and os.environ.get("LEONE_NO_DELTA_MMA", "0") != "1"):
+            image = self.mixers.leone_gated_delta_mma_image(dim)
+            if image > 0:
+                # prompt portions in bfloat16 runs: 16 tokens at a time on tensor cores
+                groups = int(sum(-(-int(q) // 16) for q in ctx.q_lens))
+                images = self._scratch("delta_images", groups * heads, image, torch.uint8)
+                self.launches += 2
+                _check(self.mixers.leone_gated_delta_mma(
+                    _ptr(act), act.stride(0), q_off, k_off, v_off, _dt(raw.dtype), _ptr(raw), raw.stride(0), a_off, b_off,
+                    _ptr(z), 0 if z is None else z.stride(0), _ptr(a_log), _ptr(dt_bias), c_float(q_scale), _ptr(out),
+                    out.stride(0), _ptr(state), _ptr(ctx.q_start), _ptr(ctx.slot_ids), ctx.n_seqs, heads, kv_heads, dim, vdim,
+                    state.shape[0], _ptr(images), groups, _ptr(ctx.status), self._stream()), "gated_delta (tensor cores)")
+                return
         self.launches += 1
         _check(self.mixers.leone_gated_delta(
             _ptr(act), act.stride(0), q_off, k_off, v_off, _dt(raw.dtype), _ptr(raw), raw.stride(0), a_off, b_off,

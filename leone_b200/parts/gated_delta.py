@@ -139,7 +139,12 @@ class GatedDeltaRule(Mixer):
         return (self.cols * self.hidden + self.hidden * self.hv + self.z_cols * (self.a_rows + self.g_rows)) * self.rt.dtype.itemsize
 
     def scratch_bytes(self, max_tokens):
-        return max_tokens * ((self.cols + self.conv_cols + self.z_cols + self.hv) * 4 + self.hv * self.rt.dtype.itemsize)
+        rows = max_tokens * ((self.cols + self.conv_cols + self.z_cols + self.hv) * 4 + self.hv * self.rt.dtype.itemsize)
+        if self.rt.dtype == torch.float32 or self.dim > 128:
+            return rows
+        # prompt portions on tensor cores: what 16 tokens of a head bring, as bfloat16 terms (csrc/gated_delta_mma.cu)
+        padded = 64 if self.dim <= 64 else 128
+        return rows + min(max_tokens, max_tokens // 16 + 256) * self.heads * (192 * (padded + 8) + 3072 + 4 * padded)
 
     def load_transient_bytes(self):
         return self.cols * self.hidden * self.rt.dtype.itemsize

@@ -260,7 +260,7 @@ def test_residual_stream_after_every_layer_on_the_gpu(which):
 
 
 @pytest.mark.gpu
-@pytest.mark.parametrize("switch", ["LEONE_NO_SSD_MMA", "LEONE_NO_TENSOR_CORES", "LEONE_NO_MASKED_MMA"])
+@pytest.mark.parametrize("switch", ["LEONE_NO_SSD_MMA", "LEONE_NO_DELTA_MMA", "LEONE_NO_TENSOR_CORES", "LEONE_NO_MASKED_MMA"])
 @pytest.mark.parametrize("which", ["C", "D"])
 def test_bfloat16_kernel_switches(which, switch, monkeypatch):
     """With a bfloat16 kernel's switch thrown its any-size form runs, and the same traces still agree
@@ -533,46 +533,65 @@ def test_ssd_kernels_against_the_plain_recurrence(heads, groups, n_state, vdim, 
 
 
 @pytest.mark.gpu
-@pytest.mark.parametrize("heads,kv_heads,dim,vdim", [(4, 2, 12, 20), (1, 1, 36, 12), (6, 3, 10, 14), (2, 1, 64, 64), (2, 2, 128, 128),
-                                                     (3, 1, 144, 24), (1, 1, 300, 40), (8, 2, 32, 33), (1, 1, 512, 64)])
-def test_delta_rule_kernel_with_channel_decays(heads, kv_heads, dim, vdim):
-    """The recurrence's kernel alone, every register form of it, with a decay per key channel: three sequences in steps
-    of unequal sizes with the state carried in slots that are not in order."""
+@pytest.mark.parametrize("per_channel", [True, False])
+@pytest.mark.parametrize("heads,kv_heads,dim,vdim,strong", [
+    (4, 2, 12, 20, 0.0), (1, 1, 36, 12, 0.0), (6, 3, 10, 14, 0.0), (2, 1, 64, 64, 0.0), (2, 2, 128, 128, 0.0), (3, 1, 144, 24, 0.0),
+    (1, 1, 300, 40, 0.0), (8, 2, 32, 33, 0.0), (1, 1, 512, 64, 0.0), (2, 1, 100, 72, 0.0), (1, 1, 65, 1, 0.0),
+    # decays so strong that sixteen of them together leave nothing (and single ones that leave next to nothing), or none
+    (2, 1, 64, 64, 4.0), (2, 2, 128, 40, 30.0), (3, 1, 48, 32, -12.0)])
+def test_delta_rule_kernels_against_the_plain_recurrence(heads, kv_heads, dim, vdim, strong, per_channel, monkeypatch):
+    """The recurrence's kernels alone in every form (the walk's register forms, tensor cores), with a decay per key channel
+    and with one per head: three sequences in steps of unequal sizes with the state carried in slots that are not in
+    order."""
     from leone_b200.ops.cuda import CudaOps
     g = torch.Generator().manual_seed(dim + vdim)
-    lengths, slots = [57, 3, 21], [2, 0, 3]
+    lengths, slots = [277, 3, 85], [2, 0, 3]
     qk, hv = kv_heads * dim, heads * vdim
     acts = [torch.randn(n, 2 * qk + hv, generator=g) for n in lengths]
-    raws = [(torch.randn(n, heads + 3, generator=g) * 2).to(torch.bfloat16) for n in lengths]
-    zs = [torch.randn(n, heads * dim + 5, generator=g) * 2 - 1 for n in lengths]
-    a_log = torch.randn(heads, generator=g) * 0.5
-    cuts = [[40, 1, 1, 2, 13], [1, 2], [2, 1, 18]]
-    for raw_dtype in (torch.float32, torch.bfloat16):
-        ops = CudaOps("cuda:0", torch.float32)
-        state = torch.randn(4, heads, dim, vdim, generator=g).cuda()
+    for a in acts:
+        # every key is like the one before it, so that the corrections matter
+        for t in range(1, len(a)):
+            a[t, qk:2 * qk] = 0.7 * a[t - 1, qk:2 * qk] + 0.5 * a[t, qk:2 * qk]
+    raws = [(torch.randn(n, 2 * heads + 3, generator=g) * 2).to(torch.bfloat16) for n in lengths]
+    zs = [torch.randn(n, heads * dim + 5, generator=g) * 2 - 1 + strong for n in lengths]
+    a_log, dt_bias = torch.randn(heads, generator=g) * 0.5, torch.randn(heads, generator=g) - 2 + strong
+    cuts = [[200, 1, 1, 2, 73], [1, 2], [2, 1, 82]]
+    rep = heads // kv_heads
+    want, states = [], []
+    for s, n in enumerate(lengths):
+        a, r = acts[s].double(), raws[s].double()
+        q = (plain.unit(a[:, :qk].view(n, kv_heads, dim)) * dim ** -0.5).repeat_interleave(rep, dim=1)
+        k = plain.unit(a[:, qk:2 * qk].view(n, kv_heads, dim)).repeat_interleave(rep, dim=1)
+        z = zs[s][:, :heads * dim].double().view(n, heads, dim) if per_channel else (r[:, 3:3 + heads] + dt_bias.double())[:, :, None].expand(n, heads, dim)
+        decay = torch.exp(-torch.exp(a_log.double())[None, :, None] * plain.softplus(z))
+        o, S = plain.delta_recurrence(q, k, a[:, 2 * qk:].view(n, heads, vdim), decay, torch.sigmoid(r[:, 3 + heads:]))
+        want.append(o.reshape(n, hv))
+        states.append(S)
+    for dtype, raw_dtype, switch, tol in ((torch.float32, torch.float32, "0", 3e-5), (torch.bfloat16, torch.bfloat16, "1", 3e-5),
+                                          (torch.bfloat16, torch.bfloat16, "0", 1e-4), (torch.bfloat16, torch.float32, "0", 1e-4)):
+        monkeypatch.setenv("LEONE_NO_DELTA_MMA", switch)
+        ops = CudaOps("cuda:0", dtype)
+        state = torch.randn(4, heads, dim, vdim, generator=g).cuda()        # what a slot held before must not matter
         state[slots] = 0.0
-        done, got = [0, 0, 0], [torch.zeros(n, hv) for n in lengths]
+        done, got = [0, 0, 0], [torch.zeros(n, hv, dtype=torch.float64) for n in lengths]
         for step in range(5):
             live = [s for s in range(3) if step < len(cuts[s])]
             q_lens = [cuts[s][step] for s in live]
             ctx, starts = _step_ctx(q_lens, [done[s] + cuts[s][step] for s in live], [slots[s] for s in live])
             act, raw, z = (torch.cat([src[s][done[s]:done[s] + cuts[s][step]] for s in live]).cuda() for src in (acts, raws, zs))
             out = torch.zeros(sum(q_lens), hv, device="cuda:0")
-            ops.gated_delta(ctx, act, raw.to(raw_dtype), out, state, a_log.cuda(), None, heads, kv_heads, dim, vdim, 0, qk, 2 * qk,
-                            0, 3, dim ** -0.5, channel_logits=z[:, :heads * dim])
+            kw = {"channel_logits": z[:, :heads * dim]} if per_channel else {}
+            ops.gated_delta(ctx, act, raw.to(raw_dtype), out, state, a_log.cuda(), None if per_channel else dt_bias.cuda(), heads,
+                            kv_heads, dim, vdim, 0, qk, 2 * qk, 3, 3 + heads, dim ** -0.5, **kw)
             assert int(ctx.status[0]) == 0
             for j, s in enumerate(live):
-                got[s][done[s]:done[s] + cuts[s][step]] = out[starts[j]:starts[j + 1]].cpu()
+                got[s][done[s]:done[s] + cuts[s][step]] = out[starts[j]:starts[j + 1]].cpu().double()
                 done[s] += cuts[s][step]
-        rep = heads // kv_heads
-        for s, n in enumerate(lengths):
-            a = acts[s].double()
-            q = (plain.unit(a[:, :qk].view(n, kv_heads, dim)) * dim ** -0.5).repeat_interleave(rep, dim=1)
-            k = plain.unit(a[:, qk:2 * qk].view(n, kv_heads, dim)).repeat_interleave(rep, dim=1)
-            decay = torch.exp(-torch.exp(a_log.double())[None, :, None] * plain.softplus(zs[s][:, :heads * dim].double()).view(n, heads, dim))
-            o, S = plain.delta_recurrence(q, k, a[:, 2 * qk:].view(n, heads, vdim), decay, torch.sigmoid(raws[s][:, 3:].double()))
-            assert float((got[s].double() - o.reshape(n, hv)).abs().max()) <= 3e-5 * float(o.abs().max()), s
-            assert float((state[slots[s]].cpu().double() - S).abs().max()) <= 3e-5 * float(S.abs().max())
+        for s in range(3):
+            err = float((got[s] - want[s]).abs().max()) / float(want[s].abs().max())
+            assert err <= tol, (dtype, switch, s, err)
+            serr = float((state[slots[s]].cpu().double() - states[s]).abs().max()) / float(states[s].abs().max())
+            assert serr <= tol, (dtype, switch, s, "state", serr)
 
 
 @pytest.mark.gpu
