@@ -200,7 +200,7 @@ gated_delta_kernel(const float* __restrict__ act, int lda, int q_off, int k_off,
   }
 }
 
-// gate_act: 0 sigmoid, 1 silu.  One block per token, a warp per head in turn.
+// gate_act: 0 sigmoid, 1 silu.  A warp per (token, head).
 template <typename T, typename TW>
 __global__ void __launch_bounds__(256)
 group_gate_norm_kernel(const float* __restrict__ o, int ldo, int heads, int vdim, const TW* __restrict__ w,
@@ -208,7 +208,8 @@ group_gate_norm_kernel(const float* __restrict__ o, int ldo, int heads, int vdim
   pdl_trigger();
   pdl_wait();
   const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  for (int h = warp; h < heads; h += 8) {
+  const int h = blockIdx.y * 8 + warp;
+  if (h < heads) {
     const float* row = o + (size_t)t * ldo + (size_t)h * vdim;
     float ss = 0.f;
     for (int c = lane; c < vdim; c += 32) ss = fmaf(row[c], row[c], ss);
@@ -233,12 +234,13 @@ using namespace leone;
 // act: fp32 [n_tokens, lda] with the activations of q and k (kv_heads x dim each) and v (heads x vdim) at
 // the given column offsets; raw: [n_tokens, ldr] in `raw_dtype` with one a and one b per head at theirs.
 // zs: fp32 [n_tokens, ldz], head h's decay logits (bias added) at columns h * dim, or null (a decay per head from a).
-// out: fp32 [n_tokens, ldo], head h at columns h * vdim.  state: fp32 [n_slots, heads, dim, vdim].
+// out: fp32 [n_tokens, ldo], head h at columns h * vdim.  state: fp32 [n_slots, heads, dim, vdim].  one_token: every sequence
+// of the step brings one token (only the choice of form depends on it).
 extern "C" int leone_gated_delta(const float* act, int lda, int q_off, int k_off, int v_off, int raw_dtype,
                                  const void* raw, int ldr, int a_off, int b_off, const float* zs, int ldz, const float* a_log, const float* dt_bias, float q_scale,
                                  float* out, int ldo, float* state, const int* q_start, const int* slot_ids,
-                                 int n_seqs, int heads, int kv_heads, int dim, int vdim, int n_slots, int* status,
-                                 cudaStream_t stream) {
+                                 int n_seqs, int heads, int kv_heads, int dim, int vdim, int n_slots, int one_token,
+                                 int* status, cudaStream_t stream) {
   if (n_seqs <= 0) return 0;
   if (heads <= 0 || kv_heads <= 0 || heads % kv_heads != 0 || dim <= 0 || vdim <= 0 || dim > 512 || heads > 65535 ||
       n_seqs > 65535)
@@ -268,6 +270,9 @@ extern "C" int leone_gated_delta(const float* act, int lda, int q_off, int k_off
   // rows dealt to 16 lanes from 33 rows on: a token's cost is the latency of its chain of sums and shuffles,
   // not its multiply-adds (dim 128: 0.48 us a token with 16 lanes a column, 0.59 with 4), and two columns a warp
   // give a prompt of one sequence 8 blocks a head
+  // (one token a sequence: whole rows of the state are read and written, so that more columns a block matter)
+  if (one_token && dim > 32 && dim <= 64) DELTA(16, 4)
+  if (one_token && dim > 64 && dim <= 128) DELTA(32, 4)
   if (dim <= 16) DELTA(4, 4)
   if (dim <= 32) DELTA(8, 4)
   if (dim <= 64) DELTA(4, 16)
@@ -286,7 +291,7 @@ extern "C" int leone_group_gate_norm(int dtype, const float* o, int ldo, int n_t
   if (n_tokens <= 0) return 0;
   if (heads <= 0 || vdim <= 0) return kRefusedSize;
 #define GGN(T, TW)                                                                                                  \
-  return launch_kernel(group_gate_norm_kernel<T, TW>, dim3(n_tokens), dim3(256), 0, stream, o, ldo, heads, vdim,    \
+  return launch_kernel(group_gate_norm_kernel<T, TW>, dim3(n_tokens, (heads + 7) / 8), dim3(256), 0, stream, o, ldo, heads, vdim,    \
                        (const TW*)w, gate, ldg, gate_act, (T*)out, ldout, eps)
   if (dtype == 0 && w_dtype == 0) GGN(float, float);
   if (dtype == 1 && w_dtype == 0) GGN(__nv_bfloat16, float);

@@ -26,6 +26,10 @@ namespace leone {
 constexpr int kConvThreads = 128;
 constexpr int kMaxTaps = 16;
 
+// v * sigmoid(v); of bfloat16 inputs with the hardware's exponential and reciprocal (a few units in fp32's last place)
+template <typename TI> __device__ __forceinline__ float conv_silu(float v) { return v / (1.f + expf(-v)); }
+template <> __device__ __forceinline__ float conv_silu<__nv_bfloat16>(float v) { return __fdividef(v, 1.f + __expf(-v)); }
+
 template <typename TI, typename TO>
 __global__ void __launch_bounds__(kConvThreads)
 short_conv_kernel(const TI* __restrict__ x, int ldx, const float* __restrict__ w, const float* __restrict__ bias, float* state,
@@ -57,7 +61,7 @@ short_conv_kernel(const TI* __restrict__ x, int ldx, const float* __restrict__ w
     acc = fmaf(w[(size_t)c * taps + j], v, acc);
   }
   if (add_input & 1) acc += to_float<TI>(x[(size_t)t * ldx + c]);
-  if (add_input & 2) acc = acc / (1.f + expf(-acc));
+  if (add_input & 2) acc = conv_silu<TI>(acc);
   out[(size_t)t * ldo + c] = from_float<TO>(acc);
   if (update_state && taps > 1 && local == 0 && q_start[s + 1] - q_start[s] == 1) {
     for (int r = 0; r + 2 < taps; ++r) st[(size_t)r * channels + c] = st[(size_t)(r + 1) * channels + c];
@@ -70,6 +74,7 @@ short_conv_kernel(const TI* __restrict__ x, int ldx, const float* __restrict__ w
 // are loaded once (V = 4: as 16- or 8-byte vectors) and every output is formed from registers; a tile
 // that spans sequences falls back to token-by-token.  kT is the most taps the form takes (its
 // register arrays are sized by it).  Per channel the sum is the one of short_conv_kernel, in the same order.
+// kExact: taps == kT (with four taps and V = 4 a channel's weights are one vector).
 constexpr int kConvTile = 8;
 
 template <typename T, int V> struct ConvVec;
@@ -105,22 +110,31 @@ template <> struct ConvVec<__nv_bfloat16, 4> {
   }
 };
 
-template <typename TI, typename TO, int V, int kT>
+template <typename TI, typename TO, int V, int kT, bool kExact>
 __global__ void __launch_bounds__(kConvThreads)
 short_conv_tile_kernel(const TI* __restrict__ x, int ldx, const float* __restrict__ w, const float* __restrict__ bias,
                        const float* __restrict__ state,
                        TO* __restrict__ out, int ldo, const int* __restrict__ q_start,
                        const int* __restrict__ seq_of_token, const int* __restrict__ slot_ids, int n_tokens, int channels,
-                       int taps, int add_input, int n_seqs, int n_slots, int* status) {
+                       int n_taps, int add_input, int n_seqs, int n_slots, int* status) {
   pdl_trigger();
+  const int taps = kExact ? kT : n_taps;
   const int t0 = blockIdx.x * kConvTile, c = (blockIdx.y * kConvThreads + threadIdx.x) * V;
   if (c >= channels) return;
   // the weights are not written during a step: fetched before the wait for the kernel ahead
   float wt[kT][V];
+  if (kExact && kT == 4 && V == 4) {               // (rows of w on 16-byte boundaries)
 #pragma unroll
-  for (int j = 0; j < kT; ++j)
+    for (int e = 0; e < V; ++e) {
+      const float4 r = *reinterpret_cast<const float4*>(w + (size_t)(c + e) * 4);
+      wt[0][e] = r.x, wt[1 % kT][e] = r.y, wt[2 % kT][e] = r.z, wt[3 % kT][e] = r.w;
+    }
+  } else {
 #pragma unroll
-    for (int e = 0; e < V; ++e) wt[j][e] = j < taps ? w[(size_t)(c + e) * taps + j] : 0.f;
+    for (int j = 0; j < kT; ++j)
+#pragma unroll
+      for (int e = 0; e < V; ++e) wt[j][e] = j < taps ? w[(size_t)(c + e) * taps + j] : 0.f;
+  }
   float b0[V];
 #pragma unroll
   for (int e = 0; e < V; ++e) b0[e] = bias != nullptr ? bias[c + e] : 0.f;
@@ -177,7 +191,7 @@ short_conv_tile_kernel(const TI* __restrict__ x, int ldx, const float* __restric
         }
         if (add_input & 2) {
 #pragma unroll
-          for (int e = 0; e < V; ++e) acc[e] = acc[e] / (1.f + expf(-acc[e]));
+          for (int e = 0; e < V; ++e) acc[e] = conv_silu<TI>(acc[e]);
         }
         ConvVec<TO, V>::store(out + (size_t)(t0 + i) * ldo + c, acc);
       }
@@ -207,7 +221,7 @@ short_conv_tile_kernel(const TI* __restrict__ x, int ldx, const float* __restric
         acc = fmaf(w[(size_t)(c + e) * taps + j], u, acc);
       }
       if (add_input & 1) acc += to_float<TI>(x[(size_t)t * ldx + c + e]);
-      if (add_input & 2) acc = acc / (1.f + expf(-acc));
+      if (add_input & 2) acc = conv_silu<TI>(acc);
       out[(size_t)(t * (size_t)ldo) + c + e] = from_float<TO>(acc);
     }
   }
@@ -519,12 +533,16 @@ extern "C" int leone_short_conv(int in_dtype, int out_dtype, const void* x, int 
   const dim3 vec_grid(tile_grid.x, (channels / 4 + kConvThreads - 1) / kConvThreads);
 #define LAUNCH(TI, TO)                                                                                              \
   {                                                                                                                 \
+    if (vec && taps == 4 && ((uintptr_t)w & 15) == 0)                                                               \
+      return launch_kernel(short_conv_tile_kernel<TI, TO, 4, 4, true>, vec_grid, dim3(kConvThreads), 0, stream,     \
+                           (const TI*)x, ldx, w, bias, state, (TO*)out, ldo, q_start, seq_of_token, slot_ids, n_tokens,  \
+                           channels, taps, add_input, n_seqs, n_slots, status);                                     \
     if (vec)                                                                                                        \
-      return launch_kernel(short_conv_tile_kernel<TI, TO, 4, 4>, vec_grid, dim3(kConvThreads), 0, stream,           \
+      return launch_kernel(short_conv_tile_kernel<TI, TO, 4, 4, false>, vec_grid, dim3(kConvThreads), 0, stream,           \
                            (const TI*)x, ldx, w, bias, state, (TO*)out, ldo, q_start, seq_of_token, slot_ids, n_tokens,  \
                            channels, taps, add_input, n_seqs, n_slots, status);                                     \
     if (tiled)                                                                                                      \
-      return launch_kernel(short_conv_tile_kernel<TI, TO, 1, kMaxTaps>, tile_grid, dim3(kConvThreads), 0, stream,   \
+      return launch_kernel(short_conv_tile_kernel<TI, TO, 1, kMaxTaps, false>, tile_grid, dim3(kConvThreads), 0, stream,   \
                            (const TI*)x, ldx, w, bias, state, (TO*)out, ldo, q_start, seq_of_token, slot_ids, n_tokens,  \
                            channels, taps, add_input, n_seqs, n_slots, status);                                     \
     return launch_kernel(short_conv_kernel<TI, TO>, grid, dim3(kConvThreads), 0, stream, (const TI*)x, ldx, w,      \

@@ -190,12 +190,13 @@ grouped_gate_norm_vec_kernel(const float* __restrict__ y, int ldy, const TZ* __r
 using namespace leone;
 
 // act: `act_dtype` [n_tokens, lda] with x (heads x vdim), B and C (groups x n_state each) at their column offsets; raw:
-// `raw_dtype` [n_tokens, ldr] with one dt per head at dt_off; out: fp32 [n_tokens, ldo], D x included.
+// `raw_dtype` [n_tokens, ldr] with one dt per head at dt_off; out: fp32 [n_tokens, ldo], D x included.  one_token: every
+// sequence of the step brings one token (only the choice of form depends on it).
 extern "C" int leone_ssd(int act_dtype, const void* act, int lda, int x_off, int b_off, int c_off, int raw_dtype,
                          const void* raw, int ldr, int dt_off, const float* a_log, const float* dt_bias,
                          const float* d_skip, float* out, int ldo, float* state, const int* q_start, const int* slot_ids,
-                         int n_seqs, int heads, int groups, int n_state, int vdim, int n_slots, int* status,
-                         cudaStream_t stream) {
+                         int n_seqs, int heads, int groups, int n_state, int vdim, int n_slots, int one_token,
+                         int* status, cudaStream_t stream) {
   if (n_seqs <= 0) return 0;
   if (heads <= 0 || groups <= 0 || heads % groups != 0 || n_state <= 0 || n_state > 512 || vdim <= 0 || heads > 65535 ||
       n_seqs > 65535)
@@ -222,6 +223,7 @@ extern "C" int leone_ssd(int act_dtype, const void* act, int lda, int x_off, int
     if (raw_dtype == 0) SSD_AS(__nv_bfloat16, float, DPT, P)                 \
     SSD_AS(__nv_bfloat16, __nv_bfloat16, DPT, P)                             \
   }
+  if (one_token && n_state > 64 && n_state <= 128) SSD(32, 4)     // whole rows of the state: more columns a block
   if (n_state <= 16) SSD(4, 4)
   if (n_state <= 32) SSD(8, 4)
   if (n_state <= 64) SSD(16, 4)

@@ -1100,7 +1100,8 @@ class CudaOps:
         _check(self.mixers.leone_gated_delta(
             _ptr(act), act.stride(0), q_off, k_off, v_off, _dt(raw.dtype), _ptr(raw), raw.stride(0), a_off, b_off,
             _ptr(z), 0 if z is None else z.stride(0), _ptr(a_log), _ptr(dt_bias), c_float(q_scale), _ptr(out), out.stride(0), _ptr(state), _ptr(ctx.q_start), _ptr(ctx.slot_ids),
-            ctx.n_seqs, heads, kv_heads, dim, vdim, state.shape[0], _ptr(ctx.status), self._stream()), "gated_delta")
+            ctx.n_seqs, heads, kv_heads, dim, vdim, state.shape[0],
+            1 if ctx.decode_only else 0, _ptr(ctx.status), self._stream()), "gated_delta")
 
     def group_gate_norm(self, o, weight, gate, out, eps, heads, vdim, act="sigmoid"):
         """``out[t, h, :] = rms_norm(o[t, h, :]) * weight * act(gate[t, h, :])``: every head normed on its own,
@@ -1153,7 +1154,8 @@ class CudaOps:
         _check(self.mixers.leone_ssd(
             _dt(act.dtype), _ptr(act), act.stride(0), x_off, b_off, c_off, _dt(raw.dtype), _ptr(raw), raw.stride(0), dt_off,
             _ptr(a_log), _ptr(dt_bias), _ptr(d_skip), _ptr(out), out.stride(0), _ptr(state), _ptr(ctx.q_start),
-            _ptr(ctx.slot_ids), ctx.n_seqs, heads, groups, n_state, vdim, state.shape[0], _ptr(ctx.status), self._stream()),
+            _ptr(ctx.slot_ids), ctx.n_seqs, heads, groups, n_state, vdim, state.shape[0],
+            1 if ctx.decode_only else 0, _ptr(ctx.status), self._stream()),
             "ssd")
 
     def grouped_gate_norm(self, y, z, weight, out, eps, groups):
