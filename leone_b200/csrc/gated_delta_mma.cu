@@ -14,8 +14,8 @@
 //
 // delta_operands: a block per (16 tokens, head) makes unit vectors, decays, M, A and T and leaves k P, q P, k P_15 / P, T and A
 // as pairs of bfloat16 terms in one image in the order of the next kernel's shared memory.
-// delta_chain: a block per (32 value columns, head, sequence) walks the images.  Eight warps: two groups of 16 value columns
-// times a quarter of the state's rows each; S^T stays in fp32 accumulator fragments, which are at the same time the A
+// delta_chain: a block per (16 or 32 value columns, head, sequence) walks the images.  Four warps to 16 value columns, a
+// quarter of the state's rows each; S^T stays in fp32 accumulator fragments, which are at the same time the A
 // operand of the read-outs; the four partial read-outs of a group meet in shared memory, after which every warp forms the
 // corrections itself and moves its rows of the state.
 #include "gla_parts.cuh"
@@ -23,7 +23,7 @@
 
 namespace leone {
 
-constexpr int kDmTokens = 16, kDmThreads = 256, kDmCols = 32;
+constexpr int kDmTokens = 16, kDmThreads = 256;
 constexpr int kDmPT = kDmTokens + 8;              // bfloat16 per row of T and A
 
 struct DeltaMmaParams {
@@ -208,15 +208,16 @@ delta_operands_kernel(const DeltaMmaParams p) {
   }
 }
 
-template <int KPW, int STAGES>
-__global__ void __launch_bounds__(kDmThreads)
+// VG: groups of 16 value columns a block
+template <int KPW, int STAGES, int VG>
+__global__ void __launch_bounds__(128 * VG)
 delta_chain_kernel(const DeltaMmaParams p) {
   pdl_trigger();
   pdl_wait();
   using I = DmImage<KPW>;
   constexpr int PD = I::PD, NT = 2 * KPW;
   extern __shared__ __align__(16) unsigned char smem_raw[];
-  float4* red = reinterpret_cast<float4*>(smem_raw + STAGES * I::bytes);      // [2 column groups][4 quarters][4][32]
+  float4* red = reinterpret_cast<float4*>(smem_raw + STAGES * I::bytes);      // [VG column groups][4 quarters][4][32]
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3, mi = lane >> 3;
   const int vg = warp >> 2, ks = warp & 3;        // this warp's group of value columns and quarter of the rows
   const int h = blockIdx.y, seq = blockIdx.z, vdim = p.vdim, dim = p.dim;
@@ -235,7 +236,9 @@ delta_chain_kernel(const DeltaMmaParams p) {
     if (grp < groups) {
       const unsigned char* src = p.images + ((size_t)(first + grp) * p.heads + h) * I::bytes;
       const uint32_t dst = base + (grp % STAGES) * I::bytes;
-      for (int i = tid * 16; i < I::bytes; i += kDmThreads * 16) cp_async16_zfill(dst + i, src + i, true);
+      #pragma unroll
+      for (int i = 0; i < I::bytes; i += 128 * VG * 16)
+        if (i + tid * 16 < I::bytes) cp_async16_zfill(dst + i + tid * 16, src + i + tid * 16, true);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
@@ -243,7 +246,7 @@ delta_chain_kernel(const DeltaMmaParams p) {
   for (int i = 0; i < STAGES - 1; ++i) request(i);
 
   float* st = p.state + ((size_t)slot * p.heads + h) * (size_t)dim * vdim;
-  const int va = blockIdx.x * kDmCols + vg * 16 + g, vb = va + 8;             // this thread's value columns
+  const int va = blockIdx.x * (16 * VG) + vg * 16 + g, vb = va + 8;             // this thread's value columns
   float S[NT][4];
 #pragma unroll
   for (int n = 0; n < NT; ++n)
@@ -256,14 +259,17 @@ delta_chain_kernel(const DeltaMmaParams p) {
   const float* v_src = p.act + p.v_off + (size_t)h * vdim;
   float V[2][4];
   auto values = [&](int grp) {
+    if (ks != 0) return;
 #pragma unroll
     for (int nn = 0; nn < 2; ++nn)
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         const int t = t0 + grp * kDmTokens + nn * 8 + 2 * tq + (i & 1), v = i < 2 ? va : vb;
-        V[nn][i] = ks == 0 && t < t1 && v < vdim ? v_src[(size_t)t * p.lda + v] : 0.f;
+        V[nn][i] = t < t1 && v < vdim ? v_src[(size_t)t * p.lda + v] : 0.f;
       }
   };
+#pragma unroll
+  for (int i = 0; i < 8; ++i) V[i >> 2][i & 3] = 0.f;
   values(0);
   const uint32_t row_b = (lane & 7) + (mi >> 1) * 8, col_b = (mi & 1) * 8;    // rows are tokens read out, columns k
   for (int grp = 0; grp < groups; ++grp) {
@@ -415,24 +421,32 @@ extern "C" int leone_gated_delta_mma(const float* act, int lda, int q_off, int k
 #define OPERANDS(KPW, CH, TR)                                                                                              \
   code = launch_kernel(delta_operands_kernel<KPW, CH, TR>, dim3(n_groups, heads), dim3(kDmThreads),                       \
                        sizeof(float) * (size_t)kDmTokens * (3 * (DmImage<KPW>::DIMP + 4) + 2 * 17 + 1), stream, p)
-#define RUN(KPW, ST)                                                                                                       \
+#define RUN(KPW, ST, VG)                                                                                                     \
   do {                                                                                                                     \
     if (zs != nullptr && raw_dtype == 0) OPERANDS(KPW, true, float);                                                       \
     else if (zs != nullptr) OPERANDS(KPW, true, __nv_bfloat16);                                                            \
     else if (raw_dtype == 0) OPERANDS(KPW, false, float);                                                                  \
     else OPERANDS(KPW, false, __nv_bfloat16);                                                                              \
     if (code != 0) return code;                                                                                            \
-    constexpr size_t smem = (size_t)ST * DmImage<KPW>::bytes + 2 * 4 * 4 * 32 * sizeof(float4);                            \
+    constexpr size_t smem = (size_t)ST * DmImage<KPW>::bytes + VG * 4 * 4 * 32 * sizeof(float4);                           \
     static bool configured = false;                                                                                        \
     if (!configured) {                                                                                                     \
-      cudaFuncSetAttribute(delta_chain_kernel<KPW, ST>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);           \
+      cudaFuncSetAttribute(delta_chain_kernel<KPW, ST, VG>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);       \
       configured = true;                                                                                                   \
     }                                                                                                                      \
-    return launch_kernel(delta_chain_kernel<KPW, ST>, dim3((vdim + kDmCols - 1) / kDmCols, heads, n_seqs), dim3(kDmThreads), \
-                         smem, stream, p);                                                                                 \
+    return launch_kernel(delta_chain_kernel<KPW, ST, VG>, dim3((vdim + 16 * VG - 1) / (16 * VG), heads, n_seqs),           \
+                         dim3(128 * VG), smem, stream, p);                                                                 \
   } while (0)
-  if (dim <= 64) RUN(1, 4);
-  RUN(2, 3);
+  // a chain of groups is bound by its latency, so that few columns a block and many blocks are fastest while the SMs
+  // last (16 heads of 128: 182 us against 229); beyond, two groups of columns share the images' copies (32 heads: 272
+  // against 347)
+  const long long narrow = (long long)((vdim + 15) / 16) * heads * n_seqs;
+  if (narrow <= 148) {
+    if (dim <= 64) RUN(1, 4, 1);
+    RUN(2, 4, 1);
+  }
+  if (dim <= 64) RUN(1, 4, 2);
+  RUN(2, 3, 2);
 #undef RUN
 #undef OPERANDS
 }

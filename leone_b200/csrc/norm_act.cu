@@ -229,11 +229,18 @@ rms_norm_add_vec_kernel(float* __restrict__ dst, const float* __restrict__ a, co
   const size_t base = (size_t)blockIdx.x * width;
   const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
   float4 va[R], vb[R], vd[R];
+  // short rows: the weights are asked for with the row, so that no load stands between two sums
+  constexpr bool kAhead = R <= 2;
+  float4 wa_r[kAhead ? R : 1], wn_r[kAhead ? R : 1];
   float sa = 0.f, sb = 0.f;
 #pragma unroll
   for (int i = 0; i < R; ++i) {
     const int c = (threadIdx.x + i * blockDim.x) * 4;
     const bool in = c < width;
+    if (kAhead) {
+      wa_r[i] = in ? row_load4<TW>(w_a + c) : zero;
+      wn_r[i] = in && next_out != nullptr ? row_load4<float>(next_w + c) : zero;
+    }
     va[i] = in ? row_load4<float>(a + base + c) : zero;
     vb[i] = in && b != nullptr ? row_load4<float>(b + base + c) : zero;
     vd[i] = in && accumulate ? row_load4<float>(dst + base + c) : zero;
@@ -252,7 +259,7 @@ rms_norm_add_vec_kernel(float* __restrict__ dst, const float* __restrict__ a, co
   for (int i = 0; i < R; ++i) {
     const int c = (threadIdx.x + i * blockDim.x) * 4;
     if (c < width) {
-      const float4 wa = row_load4<TW>(w_a + c);
+      const float4 wa = kAhead ? wa_r[kAhead ? i : 0] : row_load4<TW>(w_a + c);
       float4 v = make_float4(va[i].x * ra * wa.x, va[i].y * ra * wa.y, va[i].z * ra * wa.z, va[i].w * ra * wa.w);
       if (b != nullptr) {
         const float4 wb = row_load4<TW>(w_b + c);
@@ -294,7 +301,7 @@ rms_norm_add_vec_kernel(float* __restrict__ dst, const float* __restrict__ a, co
     for (int i = 0; i < R; ++i) {
       const int c = (threadIdx.x + i * blockDim.x) * 4;
       if (c < width) {
-        const float4 wn = row_load4<float>(next_w + c);
+        const float4 wn = kAhead ? wn_r[kAhead ? i : 0] : row_load4<float>(next_w + c);
         row_store4<TR>(next_out + base + c, make_float4(va[i].x * rn * wn.x, va[i].y * rn * wn.y, va[i].z * rn * wn.z, va[i].w * rn * wn.w));
       }
     }

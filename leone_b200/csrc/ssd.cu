@@ -6,8 +6,8 @@
 //
 // x, B and C arrive as activations (after their convolution and silu), dt as a raw projection.  Everything here is
 // fp32.  The state is read from and written back to the request's state slot and the walk is token by token in the
-// same order whatever the cut; a step of one token per sequence (decode) is the same kernel.  Prompt portions of bfloat16
-// runs have a form of their own (ssd_mma.cu).
+// same order whatever the cut.  A step of one token per sequence (decode) has a form that asks for all of a head's state at
+// once; prompt portions of bfloat16 runs have one of their own (ssd_mma.cu).
 //
 // A block owns (a slice of value columns, head, sequence).  A value column's rows are dealt to P lanes (row i belongs
 // to lane part i % P), DPT rows each in registers; the sum over rows is P-lane shuffles.  Tokens are staged 16 at a time,
@@ -107,6 +107,74 @@ ssd_walk_kernel(const SsdParams p) {
   }
 }
 
+// One token a sequence (decode): a block per (head, sequence).  A thread owns four neighbouring value columns of the rows
+// r, r + R, r + 2 R, ... and asks for up to eight of its rows of the state before it touches any; the row groups' partial
+// read-outs are summed in shared memory, in order.  Rows of the state must start on 16-byte boundaries.
+constexpr int kSsdStepThreads = 256, kSsdStepAhead = 8;
+
+template <typename TA, typename TR>
+__global__ void __launch_bounds__(kSsdStepThreads)
+ssd_step_kernel(const SsdParams p) {
+  pdl_trigger();
+  pdl_wait();
+  __shared__ __align__(16) float4 part_s[kSsdStepThreads];
+  const int tid = threadIdx.x, h = blockIdx.x, s = blockIdx.y, n_state = p.n_state, vdim = p.vdim;
+  const int quads = vdim >> 2, R = kSsdStepThreads / quads, r = tid / quads, c = (tid - r * quads) * 4;
+  const int t = p.q_start[s];
+  if (t >= p.q_start[s + 1]) return;
+  const int slot = p.slot_ids[s];
+  if (slot < 0 || slot >= p.n_slots) {
+    if (tid == 0) set_status(p.status, kBadSequence, s, slot);
+    return;
+  }
+  const TA* row = reinterpret_cast<const TA*>(p.act) + (size_t)t * p.lda;
+  const TA* bc = row + (size_t)(h / (p.heads / p.groups)) * n_state;
+  const float d = ssd_step(to_float<TR>(reinterpret_cast<const TR*>(p.raw)[(size_t)t * p.ldr + p.dt_off + h]), p.dt_bias[h]);
+  const float a = expf(-expf(p.a_log[h]) * d);
+  float x[4], y[4] = {0.f, 0.f, 0.f, 0.f};
+  if (r < R) {
+#pragma unroll
+    for (int e = 0; e < 4; ++e) x[e] = to_float<TA>(row[p.x_off + (size_t)h * vdim + c + e]);
+    float* st = p.state + ((size_t)slot * p.heads + h) * (size_t)n_state * vdim + c;
+    for (int i0 = r; i0 < n_state; i0 += R * kSsdStepAhead) {
+      float4 S[kSsdStepAhead];
+      float b[kSsdStepAhead], q[kSsdStepAhead];
+#pragma unroll
+      for (int j = 0; j < kSsdStepAhead; ++j) {
+        const int i = i0 + j * R;
+        if (i < n_state) {
+          S[j] = *reinterpret_cast<const float4*>(st + (size_t)i * vdim);
+          b[j] = to_float<TA>(bc[p.b_off + i]) * d;
+          q[j] = to_float<TA>(bc[p.c_off + i]);
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < kSsdStepAhead; ++j) {
+        const int i = i0 + j * R;
+        if (i < n_state) {
+          S[j].x = fmaf(a, S[j].x, b[j] * x[0]);
+          S[j].y = fmaf(a, S[j].y, b[j] * x[1]);
+          S[j].z = fmaf(a, S[j].z, b[j] * x[2]);
+          S[j].w = fmaf(a, S[j].w, b[j] * x[3]);
+          y[0] = fmaf(S[j].x, q[j], y[0]);
+          y[1] = fmaf(S[j].y, q[j], y[1]);
+          y[2] = fmaf(S[j].z, q[j], y[2]);
+          y[3] = fmaf(S[j].w, q[j], y[3]);
+          *reinterpret_cast<float4*>(st + (size_t)i * vdim) = S[j];
+        }
+      }
+    }
+    part_s[r * quads + (c >> 2)] = make_float4(y[0], y[1], y[2], y[3]);
+  }
+  __syncthreads();
+  const float* part = reinterpret_cast<const float*>(part_s);
+  for (int v = tid; v < vdim; v += kSsdStepThreads) {
+    float sum = 0.f;
+    for (int g = 0; g < R; ++g) sum += part[g * vdim + v];
+    p.out[(size_t)t * p.ldo + (size_t)h * vdim + v] = fmaf(p.d_skip[h], to_float<TA>(row[p.x_off + (size_t)h * vdim + v]), sum);
+  }
+}
+
 // One block per (token, group): out = (y * silu(z)) / rms over the group * w.
 template <typename TZ, typename T>
 __global__ void __launch_bounds__(256)
@@ -191,7 +259,7 @@ using namespace leone;
 
 // act: `act_dtype` [n_tokens, lda] with x (heads x vdim), B and C (groups x n_state each) at their column offsets; raw:
 // `raw_dtype` [n_tokens, ldr] with one dt per head at dt_off; out: fp32 [n_tokens, ldo], D x included.  one_token: every
-// sequence of the step brings one token (only the choice of form depends on it).
+// sequence of the step brings one token.
 extern "C" int leone_ssd(int act_dtype, const void* act, int lda, int x_off, int b_off, int c_off, int raw_dtype,
                          const void* raw, int ldr, int dt_off, const float* a_log, const float* dt_bias,
                          const float* d_skip, float* out, int ldo, float* state, const int* q_start, const int* slot_ids,
@@ -204,6 +272,14 @@ extern "C" int leone_ssd(int act_dtype, const void* act, int lda, int x_off, int
   if ((act_dtype | 1) != 1 || (raw_dtype | 1) != 1) return kRefusedDtype;
   SsdParams p = {act, lda, x_off, b_off, c_off, raw, ldr, dt_off, a_log, dt_bias, d_skip, out, ldo, state, q_start,
                  slot_ids, n_seqs, heads, groups, n_state, vdim, n_slots, status, 0, nullptr, nullptr};
+  if (one_token && vdim % 4 == 0 && vdim <= 4 * kSsdStepThreads && ((uintptr_t)state & 15) == 0) {
+#define STEP(TA, TR) return launch_kernel(ssd_step_kernel<TA, TR>, dim3(heads, n_seqs), dim3(kSsdStepThreads), 0, stream, p)
+    if (act_dtype == 0 && raw_dtype == 0) STEP(float, float);
+    if (act_dtype == 0) STEP(float, __nv_bfloat16);
+    if (raw_dtype == 0) STEP(__nv_bfloat16, float);
+    STEP(__nv_bfloat16, __nv_bfloat16);
+#undef STEP
+  }
 #define SSD_AS(TA, TR, DPT, P)                                                                                        \
   {                                                                                                                   \
     constexpr int cols = (32 / P) * (kSsdThreads / 32);                                                               \
@@ -223,7 +299,6 @@ extern "C" int leone_ssd(int act_dtype, const void* act, int lda, int x_off, int
     if (raw_dtype == 0) SSD_AS(__nv_bfloat16, float, DPT, P)                 \
     SSD_AS(__nv_bfloat16, __nv_bfloat16, DPT, P)                             \
   }
-  if (one_token && n_state > 64 && n_state <= 128) SSD(32, 4)     // whole rows of the state: more columns a block
   if (n_state <= 16) SSD(4, 4)
   if (n_state <= 32) SSD(8, 4)
   if (n_state <= 64) SSD(16, 4)
